@@ -60,13 +60,17 @@ typedef enum smc_status {
 
 /* QuantDType values (SharpMind.Core/Quantization/QuantDType.cs:2-18) */
 enum { SMC_Q8_0 = 8, SMC_Q4_K = 12, SMC_Q6_K = 14 };
+/* Dense formats, in GGUF's numbering.  A SMC_BF16 weight is [N, K] bfloat16 row-major; SMC_F32 names fp32 activations. */
+enum { SMC_F32 = 0, SMC_BF16 = 30 };
 
 /* How a quantized matmul treats its activations. */
 enum {
     SMC_ACT_F32 = 0,  /* fp32 activations x dequantised weights, fp32 accumulate (reference semantics) */
     SMC_ACT_Q8 = 1,   /* activations quantised to Q8_0 blocks on device, exact int32 block dots */
-    SMC_REF_ORDER = 2 /* fp32 activations, the scalar tier's own operation order and fp64 running
+    SMC_REF_ORDER = 2, /* fp32 activations, the scalar tier's own operation order and fp64 running
                          sum: bit-identical to VecDot*_Scalar; any K; needs the raw layout kept */
+    SMC_ACT_BF16 = 3  /* SMC_BF16 weights only: activations rounded to bfloat16, products summed in fp32 on the tensor cores
+                         (SMC_ACT_F32 over such a weight multiplies fp32 activations in fp32) */
 };
 
 /* smc_weight_register flags */
@@ -409,6 +413,11 @@ SMC_API int smc_forward_last_logits(smc_ctx *ctx, smc_model *model, const int *d
  * it are never read and are overwritten by the next append. */
 SMC_API int smc_forward_logits(smc_ctx *ctx, smc_model *model, const int *d_tokens, int seqLen, int seq, int pos, int mode,
                                float *d_logits, int *d_argmax, float *d_hidden, void *stream);
+/* The same pass with the LM head applied to chosen rows only: d_rows [n_rows] (device) names places among the `seqLen`
+ * tokens, d_logits is [n_rows, vocab] in that order.  n_rows may be 0 (d_rows and d_logits are then not read): the tokens
+ * only enter the cache.  No counterpart in the reference, whose forward passes return the last row or every row. */
+SMC_API int smc_forward_rows(smc_ctx *ctx, smc_model *model, const int *d_tokens, int seqLen, int seq, int pos, int mode,
+                             const int *d_rows, int n_rows, float *d_logits, int *d_argmax, void *stream);
 /* The acceptance rule of a verification round (MedusaGenerator.cs:262-283): d_draft [heads + 1] holds the model's own
  * greedy token followed by the heads' guesses, d_argmax [heads + 1] the greedy pick after each of them;
  * *d_accepted = 1 + the longest prefix i < heads with d_argmax[i] == d_draft[i + 1]. */
@@ -419,6 +428,81 @@ SMC_API int smc_verify_greedy_dev(smc_ctx *ctx, const int *d_argmax, const int *
  * in the reference's order; the LM head runs in SMC_REF_ORDER when the weight kept its GGUF copy, else SMC_ACT_F32. */
 SMC_API int smc_medusa_predict_dev(smc_ctx *ctx, const float *d_hidden, const float *d_head_w, const float *d_head_b, int k,
                                    int hidden, const smc_weight *lm_head, float *d_work, int *d_tokens, void *stream);
+
+/* ---- layered decoders ---------------------------------------------------------------------------
+ * A decoder described layer by layer: every layer names its sequence mixer, the mixer's own sizes and its feed-forward.
+ * No counterpart in the reference (its architectures share one block, Arch/DecoderArch.cs); the model object answers to
+ * the same entry points as the one above: smc_decode_step, smc_forward_last_logits, smc_forward_logits,
+ * smc_forward_rows, smc_model_destroy.
+ *
+ * Layer:  x <- norm(alpha x + mixer(x));  x <- norm(alpha x + ffn(x)), both norms RMS norms whose weight vector is stored
+ * as an offset from one (x / rms * (1 + w)).  x is fp32 throughout.  The logits are norm(x) times the embedding table.
+ * Weights are SMC_BF16 handles, vectors fp32 device pointers; layers may share handles, each has its own cache or state.
+ *
+ * act_dtype SMC_BF16: activations between the matmuls and the latent cache are bfloat16 (mode SMC_ACT_BF16); SMC_F32:
+ * everything is fp32 (mode SMC_ACT_F32).  Norms, rotations, scores, softmax, recurrences and x are fp32 in both.
+ *
+ * A sequence owns slot `seq` of every layer: a latent layer keeps a ring of the last window - 1 + max_chunk positions
+ * (compressed key/value row and rotated key part), a state-space layer its fp32 state and the convolution's last inputs.
+ * Position 0 starts a sequence over.  A recurrence has no way back: `pos` must be the number of tokens the slot holds
+ * (SMC_E_RANGE otherwise).  smc_decode_step with pos = SMC_POS_NEXT takes each slot's next position from the device,
+ * so that a captured CUDA graph of the step can be replayed token after token. */
+enum { SMC_MIX_LATENT = 1, SMC_MIX_MAMBA2 = 2 };
+#define SMC_POS_NEXT (-1)
+/* Rotation angles p * f_i over pairs (i, i + dims/2), f_i = base^(-2i/dims).  factor > 0: YaRN, frequencies whose
+ * wavelength exceeds the `original` context are divided by `factor`, with a ramp between the dimensions that turn `fast`
+ * and `slow` times over it; cosine and sine are scaled by 0.1 ln(factor) + 1. */
+typedef struct smc_rotation {
+    int dims;
+    double base, factor, original, fast, slow;
+} smc_rotation;
+typedef struct smc_layer_desc {
+    int mixer;                /* SMC_MIX_* */
+    int heads, vdim;          /* both mixers: heads and value width per head */
+    /* SMC_MIX_LATENT: queries and keys of dim unrotated + rot_dim rotated elements, keys and values rebuilt from a latent
+     * of kv_rank.  window > 0: position i sees i - window + 1 .. i. */
+    int dim, rot_dim, q_rank, kv_rank, window;
+    float scale;
+    smc_rotation rot;
+    const smc_weight *w_down; /* [q_rank + kv_rank + rot_dim, hidden]: query latent, key/value latent, rotated key part */
+    const smc_weight *w_uq;   /* [heads * (dim + rot_dim), q_rank] */
+    const smc_weight *w_ukv;  /* [heads * dim + heads * vdim, kv_rank]: keys of every head, then values */
+    const float *q_norm, *kv_norm, *sink; /* [q_rank], [kv_rank], [heads] (sink may be null) */
+    /* SMC_MIX_MAMBA2: heads states of [state, vdim], B and C shared by heads / groups heads, a causal convolution of
+     * `conv` taps, the output gated by SiLU(z) and normed in norm_groups parts. */
+    int state, groups, conv, norm_groups;
+    const smc_weight *w_in;   /* [2 heads vdim + 2 groups state + heads, hidden]: z, x, B, C, dt */
+    const float *conv_w, *conv_b, *dt_bias, *a_log, *d_skip, *mix_norm;
+    const smc_weight *w_out;  /* [hidden, heads * vdim] */
+    /* feed-forward down(SiLU(gate x) * up x); ffn = 0: none */
+    int ffn;
+    const smc_weight *w_gu;   /* [2 ffn, hidden] woven by smc_weight_interleave_rows */
+    const smc_weight *w_ffn_down;
+    const float *norm1, *norm2; /* [hidden] */
+} smc_layer_desc;
+typedef struct smc_layered_desc {
+    int n_layers, hidden, vocab, max_seq, max_chunk, act_dtype;
+    float eps, alpha;
+    const smc_layer_desc *layers;
+    const smc_weight *embedding; /* [vocab, hidden], also the LM head */
+    const float *final_norm;
+} smc_layered_desc;
+SMC_API int smc_model_create_layered(smc_ctx *ctx, const smc_layered_desc *desc, int max_batch, smc_model **out);
+/* Tokens of sequence slot `seq` a layered model holds, -1 when only the device knows (after SMC_POS_NEXT steps).
+ * smc_model_seq_reset forgets them: the slot can be used for another sequence. */
+SMC_API int smc_model_seq_length(smc_ctx *ctx, const smc_model *m, int seq, int *length);
+SMC_API int smc_model_seq_reset(smc_ctx *ctx, smc_model *m, int seq);
+/* Copies the residual stream after every layer of the next forward passes to d_dump [n_layers, max_chunk, hidden] fp32
+ * (row t of layer l at (l * max_chunk + t) * hidden); null turns it off.  For bringing up a model and for tests. */
+SMC_API int smc_model_dump_layers(smc_ctx *ctx, smc_model *m, float *d_dump);
+/* Cosine and sine tables [maxSeq, rot.dims / 2] of `rot`, computed in double on the host; beside smc_rope_tables. */
+SMC_API int smc_rope_tables_yarn(smc_ctx *ctx, const smc_rotation *rot, int maxSeq, float *d_cos, float *d_sin);
+/* x = norm(alpha x + y) with norm(v)_i = v_i / rms(v) * (w_offset + w_i); y may be null.  d_x16 (may be null) also
+ * receives the rows in bfloat16.  The post-norm form of smc_add_rmsnorm_dev. */
+SMC_API int smc_scaled_add_rmsnorm_dev(smc_ctx *ctx, float *d_x, const float *d_y, const float *d_w, void *d_x16, int rows, int n,
+                                       float alpha, float w_offset, float eps, void *stream);
+/* Rows of a SMC_BF16 table as fp32: out[i] = row tokens[i]; beside smc_embed_q8_0_dev. */
+SMC_API int smc_embed_bf16_dev(smc_ctx *ctx, const smc_weight *table, const int *d_tokens, int count, float *d_out, void *stream);
 
 /* One activation row whose elementwise producer rides in the matmul's staging (SMC_ACT_Q8 arithmetic, weights that
  * the one-row bulk-copy kernel takes: registered with SMC_W_REPACK, K % 1024 == 0 for Q8_0 / K % 2048 == 0 for the

@@ -120,6 +120,14 @@ SIGNATURES = {
     "smc_copy_to_device": (c_int, [c_void_p, c_void_p, c_void_p, C.c_size_t, c_void_p]),
     "smc_copy_to_host": (c_int, [c_void_p, c_void_p, c_void_p, C.c_size_t, c_void_p]),
     "smc_forward_logits": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p]),
+    "smc_forward_rows": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p]),
+    "smc_model_create_layered": (c_int, [c_void_p, c_void_p, c_int, _pp]),
+    "smc_model_seq_length": (c_int, [c_void_p, c_void_p, c_int, C.POINTER(c_int)]),
+    "smc_model_seq_reset": (c_int, [c_void_p, c_void_p, c_int]),
+    "smc_model_dump_layers": (c_int, [c_void_p, c_void_p, c_void_p]),
+    "smc_rope_tables_yarn": (c_int, [c_void_p, c_void_p, c_int, c_void_p, c_void_p]),
+    "smc_scaled_add_rmsnorm_dev": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_float, c_void_p]),
+    "smc_embed_bf16_dev": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p]),
     "smc_verify_greedy_dev": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p]),
     "smc_medusa_predict_dev": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p]),
     "smc_kv_append_dev": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,

@@ -54,8 +54,12 @@ def build(force: bool = False, verbose: bool = False, extra: list[str] | None = 
     os.makedirs(OBJ, exist_ok=True)
     flags = NVCC_FLAGS + (extra or [])
 
+    newest_dep = max(os.path.getmtime(p) for p in _deps() + [os.path.abspath(__file__)])
+
     def compile_one(src: str) -> str:
         obj = os.path.join(OBJ, os.path.basename(src)[:-3] + ".o")
+        if not force and not extra and os.path.exists(obj) and os.path.getmtime(obj) > max(newest_dep, os.path.getmtime(src)):
+            return obj
         cmd = [nvcc(), *flags, "-c", src, "-o", obj]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode != 0:
@@ -66,10 +70,12 @@ def build(force: bool = False, verbose: bool = False, extra: list[str] | None = 
 
     with ThreadPoolExecutor(max_workers=min(8, len(sources()))) as ex:
         objs = list(ex.map(compile_one, sources()))
-    cmd = [nvcc(), "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-o", LIB, *objs]
+    part = f"{LIB}.{os.getpid()}"  # appears whole: another process may be waiting for it
+    cmd = [nvcc(), "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-o", part, *objs]
     r = subprocess.run(cmd, capture_output=True, text=True)
     if r.returncode != 0:
         raise RuntimeError(f"link failed:\n{r.stdout}\n{r.stderr}")
+    os.replace(part, LIB)
     return LIB
 
 

@@ -107,7 +107,7 @@ bool host_is_pinned(smc_ctx *ctx, const void *p)
     return pinned;
 }
 
-bool known_dtype(int dtype) { return dtype == SMC_Q8_0 || dtype == SMC_Q4_K || dtype == SMC_Q6_K; }
+bool known_dtype(int dtype) { return dtype == SMC_Q8_0 || dtype == SMC_Q4_K || dtype == SMC_Q6_K || dtype == SMC_BF16; }
 
 void free_weight(smc_weight *w)
 {
@@ -123,6 +123,7 @@ void free_weight(smc_weight *w)
 int finish_register(smc_ctx *ctx, smc_weight *w)
 {
     const int K = w->K;
+    if (w->dtype == SMC_BF16) return SMC_OK;  // row-major as it came
     const bool shape_ok = (w->dtype == SMC_Q8_0) ? (K % 32 == 0) : (K % 256 == 0);
     if ((w->flags & SMC_W_REPACK) && shape_ok) {
         int rc = smc_launch_repack(ctx, w, ctx->stream);
@@ -171,6 +172,7 @@ int64_t smc_raw_tensor_bytes(int dtype, int64_t N, int64_t K)
     case SMC_Q8_0: return N * ((K + 31) / 32) * 34;
     case SMC_Q4_K: return ((N * K + 255) / 256) * 144;
     case SMC_Q6_K: return ((N * K + 255) / 256) * 210;
+    case SMC_BF16: return N * K * 2;
     default: return -1;
     }
 }
@@ -261,7 +263,7 @@ int smc_device_status(smc_ctx *ctx, int *status)
     SMC_CUDA(ctx, cudaMemcpy(status, ctx->d_status, sizeof(int), cudaMemcpyDeviceToHost));
     if (*status) {
         SMC_CUDA(ctx, cudaMemset(ctx->d_status, 0, sizeof(int)));
-        return smc_fail(ctx, SMC_E_CUDA, "a kernel gave up a bounded wait (status %d): its outputs are invalid", *status);
+        return smc_fail(ctx, SMC_E_CUDA, "a kernel gave up a bounded wait, or (status 5) a sequence ran past max_seq (status %d): its outputs are invalid", *status);
     }
     return SMC_OK;
 }
@@ -500,11 +502,33 @@ static int qmatmul_f32_digits(smc_ctx *ctx, const float *d_in, const smc_weight 
     return smc_launch_sum3(ctx, ctx->d_digit_out, d_out, (long long)M * w->N, s);
 }
 
+// A dense bfloat16 weight: fp32 rows as they are (SMC_ACT_F32) or rounded to bfloat16 in the context's scratch first.
+static int qmatmul_dense(smc_ctx *ctx, const float *d_in, const smc_weight *w, float *d_out, int M, int mode, cudaStream_t s)
+{
+    smc_dense_out o{};
+    o.y = d_out, o.ldy = w->N;
+    if (mode == SMC_ACT_F32) return smc_launch_dense(ctx, d_in, 0, w->K, w, M, o, s);
+    if (mode != SMC_ACT_BF16) return smc_fail(ctx, SMC_E_UNSUPPORTED, "qmatmul: mode %d over a bfloat16 weight", mode);
+    std::lock_guard<std::mutex> lock(ctx->mu_scratch);
+    const size_t bytes = (size_t)M * w->K * 2;
+    if (ctx->prefill_cap < bytes) {  // growing allocates: make the first call of a new size outside stream capture
+        cudaDeviceSynchronize();
+        cudaFree(ctx->d_prefill);
+        ctx->d_prefill = nullptr, ctx->prefill_cap = 0;
+        SMC_CUDA(ctx, cudaMalloc(&ctx->d_prefill, bytes));
+        ctx->prefill_cap = bytes;
+    }
+    int rc = smc_launch_round_bf16(ctx, d_in, ctx->d_prefill, (long long)M * w->K, s);
+    if (rc) return rc;
+    return smc_launch_dense(ctx, ctx->d_prefill, 1, w->K, w, M, o, s);
+}
+
 // `gd` (row-split across GPUs): when the one-row TMA kernel runs, it also exchanges the output slice with the
 // peers and *fused is set; otherwise the caller launches the exchange after this returns.
 static int qmatmul_impl(smc_ctx *ctx, const float *d_in, const smc_weight *w, float *d_out, int M, int mode,
                         cudaStream_t s, const smc_gather_dev *gd = nullptr, bool *fused = nullptr)
 {
+    if (w->dtype == SMC_BF16) return qmatmul_dense(ctx, d_in, w, d_out, M, mode, s);
     switch (mode) {
     case SMC_REF_ORDER: return smc_launch_gemv_ref(ctx, d_in, w, d_out, M, 0, w->N, s);
     case SMC_ACT_F32:
@@ -621,7 +645,7 @@ int smc_weight_concat_rows(smc_ctx *ctx, const smc_weight *const *parts, int cou
     for (int i = 0; i < count; ++i) {
         const smc_weight *p = parts[i];
         if (!p || p->dtype != dtype || p->K != K) return smc_fail(ctx, SMC_E_SIZE_MISMATCH, "weight_concat: parts differ in dtype or K");
-        if (!p->fast) return smc_fail(ctx, SMC_E_UNSUPPORTED, "weight_concat: parts must be registered with SMC_W_REPACK");
+        if (!p->fast && dtype != SMC_BF16) return smc_fail(ctx, SMC_E_UNSUPPORTED, "weight_concat: parts must be registered with SMC_W_REPACK");
         if (dtype == SMC_Q6_K && ((long long)p->N * K / 256) % 8 != 0)
             return smc_fail(ctx, SMC_E_UNSUPPORTED, "weight_concat: a Q6_K part must hold a multiple of 2048 elements");
         raw = raw && p->d_raw != nullptr;
@@ -630,7 +654,7 @@ int smc_weight_concat_rows(smc_ctx *ctx, const smc_weight *const *parts, int cou
     if (N > INT32_MAX) return smc_fail(ctx, SMC_E_RANGE, "weight_concat: too many rows");
     SMC_CUDA(ctx, cudaSetDevice(ctx->device));
     smc_weight *w = new smc_weight();
-    w->dtype = dtype, w->N = (int)N, w->K = K, w->flags = SMC_W_REPACK | (raw ? SMC_W_KEEP_RAW : 0), w->fast = true;
+    w->dtype = dtype, w->N = (int)N, w->K = K, w->flags = SMC_W_REPACK | (raw ? SMC_W_KEEP_RAW : 0), w->fast = dtype != SMC_BF16;
     w->raw_bytes = (size_t)smc_raw_tensor_bytes(dtype, (int)N, K);
     cudaError_t e = cudaSuccess;
     // bytes per row of every array of the compute layout (rows are whole blocks when `fast`)
@@ -675,15 +699,15 @@ int smc_weight_interleave_rows(smc_ctx *ctx, const smc_weight *a, const smc_weig
     if (!ctx || !a || !b || !out) return smc_fail(ctx, SMC_E_INVALID, "weight_interleave: bad arguments");
     if (a->dtype != b->dtype || a->K != b->K || a->N != b->N)
         return smc_fail(ctx, SMC_E_SIZE_MISMATCH, "weight_interleave: the two weights differ in dtype or shape");
-    if (!a->fast || !b->fast) return smc_fail(ctx, SMC_E_UNSUPPORTED, "weight_interleave: weights must be registered with SMC_W_REPACK");
+    if (a->dtype != SMC_BF16 && (!a->fast || !b->fast)) return smc_fail(ctx, SMC_E_UNSUPPORTED, "weight_interleave: weights must be registered with SMC_W_REPACK");
     const int dtype = a->dtype, K = a->K, N = a->N;
     if (dtype == SMC_Q6_K && K % 2048) return smc_fail(ctx, SMC_E_UNSUPPORTED, "weight_interleave: Q6_K rows must be whole 2048-element units");
-    if (dtype != SMC_Q8_0 && K % 256) return smc_fail(ctx, SMC_E_UNSUPPORTED, "weight_interleave: rows must be whole blocks");
+    if (dtype != SMC_Q8_0 && dtype != SMC_BF16 && K % 256) return smc_fail(ctx, SMC_E_UNSUPPORTED, "weight_interleave: rows must be whole blocks");
     if (2LL * N > INT32_MAX) return smc_fail(ctx, SMC_E_RANGE, "weight_interleave: too many rows");
     const bool raw = a->d_raw && b->d_raw;
     SMC_CUDA(ctx, cudaSetDevice(ctx->device));
     smc_weight *w = new smc_weight();
-    w->dtype = dtype, w->N = 2 * N, w->K = K, w->flags = SMC_W_REPACK | (raw ? SMC_W_KEEP_RAW : 0), w->fast = true;
+    w->dtype = dtype, w->N = 2 * N, w->K = K, w->flags = SMC_W_REPACK | (raw ? SMC_W_KEEP_RAW : 0), w->fast = dtype != SMC_BF16;
     w->raw_bytes = (size_t)smc_raw_tensor_bytes(dtype, 2 * N, K);
     cudaError_t e = cudaSuccess;
     // row 2i of the result = row i of a, row 2i + 1 = row i of b, for every array of the compute layout
@@ -742,7 +766,7 @@ int smc_block_isums_dev(smc_ctx *ctx, const smc_q8act *a, int m, const smc_weigh
 {
     if (!ctx || !a || !w || !d_sums || m < 0 || m >= a->M || col0 < 0 || col1 > w->N || col0 > col1 || a->K != w->K)
         return smc_fail(ctx, SMC_E_INVALID, "block_isums: bad arguments");
-    if ((w->dtype == SMC_Q8_0 && w->K % 32) || (w->dtype != SMC_Q8_0 && w->K % 256))
+    if (w->dtype == SMC_BF16 || (w->dtype == SMC_Q8_0 && w->K % 32) || (w->dtype != SMC_Q8_0 && w->K % 256))
         return smc_fail(ctx, SMC_E_UNSUPPORTED, "block_isums: K must be a whole number of blocks");
     return smc_launch_block_isums(ctx, a, m, w, col0, col1, d_sums, static_cast<cudaStream_t>(stream));
 }
@@ -833,6 +857,7 @@ int smc_vecdot_host(smc_ctx *ctx, const float *input, const void *host_raw, int 
     if (rc) return rc;
     if (w->dtype != dtype || w->K != K)
         return smc_fail(ctx, SMC_E_SIZE_MISMATCH, "vecdot_host: weight was registered as dtype=%d K=%d", w->dtype, w->K);
+    if (dtype == SMC_BF16) return smc_fail(ctx, SMC_E_UNSUPPORTED, "vecdot_host: quantised formats only");
     if (col < 0 || col >= w->N) return smc_fail(ctx, SMC_E_RANGE, "vecdot_host: col %d outside [0, %d)", col, w->N);
     std::lock_guard<std::mutex> lock(ctx->mu);
     cudaSetDevice(ctx->device);

@@ -192,6 +192,88 @@ int smc_launch_sdpa_tile(smc_ctx *, const float *q, const float *k, const float 
                          int hd, float scale, int causal, int qStride, int oStride, float alibi, cudaStream_t s);
 int smc_launch_rmsnorm_row(smc_ctx *, const float *src, const float *w, float *dst, int n, float rms_inv,
                            cudaStream_t s);
+// ---- dense bfloat16 weights (smc_dense.cu) ----
+// Where a dense matmul puts its product [M, N].  Columns from `split` on (if split > 0) go to y32, fp32, stride ld32.
+// woven: the weight's rows are gate / up pairs (2i, 2i + 1) and y receives SiLU(gate) * up, N / 2 columns.
+struct smc_dense_out {
+    void *y;
+    int ldy;
+    int y_bf16;
+    float *y32;
+    int ld32, split, woven;
+};
+// x [M, K] with row stride ldx, bfloat16 (x_bf16) or fp32; fp32 rows are multiplied in fp32 on the CUDA cores.
+int smc_launch_dense(smc_ctx *, const void *x, int x_bf16, int ldx, const smc_weight *, int M, const smc_dense_out &, cudaStream_t s);
+// rows row0 .. row0 + N - 1 of the weight only
+int smc_launch_dense_rows(smc_ctx *, const void *x, int x_bf16, int ldx, const smc_weight *, int row0, int N, int M, const smc_dense_out &,
+                          cudaStream_t s);
+int smc_launch_round_bf16(smc_ctx *, const float *x, void *y, long long n, cudaStream_t s);
+// Row r of a batch: of sequence slot seq0 at position pos[seq0] + r, or (seq0 < 0) of slot r at position pos[r].
+struct smc_rows {
+    const int *pos;
+    int seq0, n;
+};
+// out = x / rms(x) * (w_offset + w) of chosen rows (row r of the output reads row rows[r], or first + r), fp32 or bfloat16
+int smc_launch_rmsnorm_gather(smc_ctx *, const float *x, const int *rows, int first, int n_rows, const float *w, void *out, int out_bf16, int n,
+                              float w_offset, float eps, cudaStream_t s);
+// embedding rows as fp32 x (and bfloat16 x16 when not null), and the step's positions: pos [slots] first positions, then
+// [slots] lengths; a step starts at pos0, or (pos0 < 0) at each slot's length
+int smc_launch_embed_bf16(smc_ctx *, const smc_weight *table, const int *tokens, int count, float *x, void *x16, int *pos, int slots, int seq0,
+                          int pos0, int max_seq, cudaStream_t s);
+// ---- latent attention (smc_latent.cu) ----
+struct smc_latent_dims {
+    int heads, dim, rot_dim, vdim, q_rank, kv_rank, window, ring;
+    float scale, eps;
+};
+struct smc_latent_bufs {          // activation buffers of a step, element type T = float or bfloat16
+    const void *down;             // [rows, q_rank + kv_rank + rot_dim]  T
+    void *cq;                     // [rows, q_rank]  T
+    const void *q;                // [rows, heads * (dim + rot_dim)]  T
+    float *qa;                    // [rows, heads, kv_rank + rot_dim]
+    float *oc;                    // [rows, heads, kv_rank]
+    void *o;                      // [rows, heads * vdim]  T
+    void *keys;                   // [window - 1 + rows, kv_rank + rot_dim]  T
+    void *kv;                     // [window - 1 + rows, heads * (dim + vdim)]  T
+    void *cache;                  // [slots, ring, kv_rank + rot_dim]  T
+};
+int smc_latent_post(smc_ctx *, const smc_latent_dims &, const smc_latent_bufs &, const smc_rows &, int bf16, const float *q_norm,
+                    const float *kv_norm, const float *cosT, const float *sinT, int max_seq, cudaStream_t s);
+int smc_latent_attend(smc_ctx *, const smc_latent_dims &, const smc_latent_bufs &, const smc_rows &, int bf16, const smc_weight *w_ukv,
+                      const float *sink, const float *cosT, const float *sinT, int max_seq, int pos0, cudaStream_t s);
+int smc_latent_reserve(smc_ctx *, const smc_latent_dims &, int max_batch);
+bool smc_latent_prefill_supported(const smc_latent_dims &);
+// ---- state-space layers (smc_ssm.cu) ----
+struct smc_ssm_dims {
+    int heads, vdim, state, groups, conv, norm_groups;
+    float eps;
+};
+struct smc_ssm_bufs {
+    const void *zx;               // [rows, ld]: z | x | B | C  T
+    int ld;
+    const float *dt_raw;          // [rows, heads]
+    void *xbc;                    // [rows, heads vdim + 2 groups state] after convolution and SiLU  T
+    float *dt;                    // [rows, heads]
+    float *y;                     // [rows, heads vdim]
+    void *o;                      // [rows, heads vdim]  T
+    void *conv_state;             // [slots, conv, channels]  T: input of position p in row p % conv
+    float *state;                 // [slots, heads, vdim, state]
+    float *work;                  // chunked pass: per chunk states and decays
+    size_t work_floats;
+};
+int smc_ssm_mix(smc_ctx *, const smc_ssm_dims &, const smc_ssm_bufs &, const smc_rows &, int bf16, const float *conv_w, const float *conv_b,
+                const float *dt_bias, const float *a_log, const float *d_skip, const float *norm, int pos0, cudaStream_t s);
+size_t smc_ssm_work_floats(const smc_ssm_dims &, int rows);
+// ---- layered models (smc_layered.cu) ----
+struct smc_layered;
+void smc_layered_free(smc_layered *);
+int smc_layered_create(smc_ctx *, const smc_layered_desc *, int max_batch, smc_layered **out);
+// all_rows: 0 last row, 1 every row, 2 rows d_rows[0 .. n_rows); seq0 < 0: one token for each of slots 0 .. count - 1
+int smc_layered_forward(smc_ctx *, smc_layered *, const int *d_tokens, int count, int seq0, int pos, int mode, int all_rows, const int *d_rows,
+                        int n_rows, float *d_logits, int *d_argmax, float *d_hidden, cudaStream_t s);
+int smc_layered_length(const smc_layered *, int seq);
+void smc_layered_reset(smc_layered *, int seq);
+void smc_layered_dump(smc_layered *, float *d_dump);
+int smc_layered_slots(const smc_layered *);
 int smc_q8act_alloc(smc_ctx *, int max_rows, int max_k, smc_q8act **out);
 void smc_q8act_free(smc_q8act *);
 

@@ -15,6 +15,7 @@
 #include "smc_common.cuh"
 
 struct smc_model {
+    smc_layered *layered = nullptr;  // a decoder described layer by layer (smc_layered.cu): the members below are then unused
     smc_model_desc d{};
     int max_batch = 0;
     int rows = 0;  // rows the activation scratch holds: max_batch, or the longest prompt chunk seen so far
@@ -44,6 +45,7 @@ namespace {
 void free_model(smc_ctx *ctx, smc_model *m)
 {
     if (!m) return;
+    smc_layered_free(m->layered);
     float *bufs[] = {m->kcache, m->vcache, m->cosT, m->sinT, m->x, m->xn, m->q, m->k, m->v, m->att, m->tmp, m->gu, m->act, m->qkv, m->x2};
     for (float *p : bufs) cudaFree(p);
     cudaFree(m->kq8), cudaFree(m->vq8), cudaFree(m->kd8), cudaFree(m->vd8);
@@ -298,9 +300,46 @@ __global__ void __launch_bounds__(256) kv_load_q8_kernel(const float *__restrict
 
 extern "C" {
 
+int smc_model_create_layered(smc_ctx *ctx, const smc_layered_desc *desc, int max_batch, smc_model **out)
+{
+    if (!ctx || !desc || !out || max_batch <= 0) return smc_fail(ctx, SMC_E_INVALID, "model_create_layered: bad arguments");
+    smc_layered *body = nullptr;
+    int rc = smc_layered_create(ctx, desc, max_batch, &body);
+    if (rc) return rc;
+    *out = new smc_model();
+    (*out)->layered = body, (*out)->max_batch = max_batch;
+    return SMC_OK;
+}
+
+int smc_model_seq_length(smc_ctx *ctx, const smc_model *m, int seq, int *length)
+{
+    if (!ctx || !m || !length) return smc_fail(ctx, SMC_E_INVALID, "seq_length: bad arguments");
+    if (!m->layered) return smc_fail(ctx, SMC_E_UNSUPPORTED, "seq_length: this model's cache keeps no length, every call names its position");
+    if (seq < 0 || seq >= m->max_batch) return smc_fail(ctx, SMC_E_RANGE, "seq_length: sequence %d outside [0, %d)", seq, m->max_batch);
+    *length = smc_layered_length(m->layered, seq);
+    return SMC_OK;
+}
+
+int smc_model_seq_reset(smc_ctx *ctx, smc_model *m, int seq)
+{
+    if (!ctx || !m) return smc_fail(ctx, SMC_E_INVALID, "seq_reset: bad arguments");
+    if (seq < 0 || seq >= m->max_batch) return smc_fail(ctx, SMC_E_RANGE, "seq_reset: sequence %d outside [0, %d)", seq, m->max_batch);
+    if (m->layered) smc_layered_reset(m->layered, seq);  // a cache that keeps no length has nothing to forget
+    return SMC_OK;
+}
+
+int smc_model_dump_layers(smc_ctx *ctx, smc_model *m, float *d_dump)
+{
+    if (!ctx || !m) return smc_fail(ctx, SMC_E_INVALID, "dump_layers: bad arguments");
+    if (!m->layered) return smc_fail(ctx, SMC_E_UNSUPPORTED, "dump_layers: layered models only");
+    smc_layered_dump(m->layered, d_dump);
+    return SMC_OK;
+}
+
 int smc_model_kv_load(smc_ctx *ctx, smc_model *m, const float *d_k, const float *d_v, int batch, int len, void *stream)
 {
     if (!ctx || !m || !d_k || !d_v || batch <= 0 || len < 0) return smc_fail(ctx, SMC_E_INVALID, "kv_load: bad arguments");
+    if (m->layered) return smc_fail(ctx, SMC_E_UNSUPPORTED, "kv_load: a layered model's state is not a K/V cache");
     if (batch > m->max_batch || len > m->d.max_seq) return smc_fail(ctx, SMC_E_RANGE, "kv_load: %d x %d exceeds the cache", batch, len);
     long long total = (long long)m->d.n_layers * batch * m->d.n_kv_heads * len * m->d.head_dim;
     if (total == 0) return SMC_OK;
@@ -446,6 +485,7 @@ int smc_model_destroy(smc_ctx *ctx, smc_model *m)
 int smc_model_kv(smc_ctx *ctx, smc_model *m, float **d_k, float **d_v)
 {
     if (!ctx || !m || !d_k || !d_v) return smc_fail(ctx, SMC_E_INVALID, "model_kv: bad arguments");
+    if (m->layered) return smc_fail(ctx, SMC_E_UNSUPPORTED, "model_kv: a layered model's state is not a K/V cache");
     if (m->kv_q8) return smc_fail(ctx, SMC_E_UNSUPPORTED, "model_kv: the model's cache holds Q8_0 rows, not floats");
     *d_k = m->kcache;
     *d_v = m->vcache;
@@ -457,6 +497,9 @@ int smc_decode_step(smc_ctx *ctx, smc_model *m, const int *d_tokens, int batch, 
 {
     if (!ctx || !m || !d_tokens || !d_logits || batch <= 0) return smc_fail(ctx, SMC_E_INVALID, "decode_step: bad arguments");
     if (batch > m->max_batch) return smc_fail(ctx, SMC_E_RANGE, "decode_step: batch %d exceeds the model's %d", batch, m->max_batch);
+    if (m->layered)
+        return smc_layered_forward(ctx, m->layered, d_tokens, batch, -1, pos, mode, 1, nullptr, 0, d_logits, d_argmax, nullptr,
+                                   static_cast<cudaStream_t>(stream));
     const smc_model_desc &d = m->d;
     if (pos < 0 || pos + 1 > d.max_seq)  // KVCache.Update throws on overflow (KVCache.cs:89-91)
         return smc_fail(ctx, SMC_E_RANGE, "KVCache overflow: position %d + seqLen 1 exceeds capacity %d", pos, d.max_seq);
@@ -569,7 +612,7 @@ int smc_decode_step(smc_ctx *ctx, smc_model *m, const int *d_tokens, int batch, 
 // all_rows == 0: Transformer.ForwardLastLogits (logits of the last position); != 0: Transformer.Forward (logits of every
 // position, [seqLen, vocab]), with the final-normed hidden states copied to d_hidden [seqLen, hidden] when given.
 static int forward_tokens(smc_ctx *ctx, smc_model *m, const int *d_tokens, int seqLen, int seq, int pos, int mode, float *d_logits,
-                          int *d_argmax, int all_rows, float *d_hidden, void *stream);
+                          int *d_argmax, int all_rows, float *d_hidden, void *stream, const int *d_rows = nullptr, int n_rows = 0);
 
 int smc_forward_last_logits(smc_ctx *ctx, smc_model *m, const int *d_tokens, int seqLen, int seq, int pos, int mode,
                             float *d_logits, int *d_argmax, void *stream)
@@ -583,11 +626,31 @@ int smc_forward_logits(smc_ctx *ctx, smc_model *m, const int *d_tokens, int seqL
     return forward_tokens(ctx, m, d_tokens, seqLen, seq, pos, mode, d_logits, d_argmax, 1, d_hidden, stream);
 }
 
-static int forward_tokens(smc_ctx *ctx, smc_model *m, const int *d_tokens, int seqLen, int seq, int pos, int mode, float *d_logits,
-                          int *d_argmax, int all_rows, float *d_hidden, void *stream)
+int smc_forward_rows(smc_ctx *ctx, smc_model *m, const int *d_tokens, int seqLen, int seq, int pos, int mode, const int *d_rows, int n_rows,
+                     float *d_logits, int *d_argmax, void *stream)
 {
-    if (!ctx || !m || !d_tokens || !d_logits || seqLen <= 0) return smc_fail(ctx, SMC_E_INVALID, "forward_last_logits: bad arguments");
+    if (n_rows < 0 || (n_rows > 0 && (!d_rows || !d_logits)) || n_rows > seqLen)
+        return smc_fail(ctx, SMC_E_INVALID, "forward_rows: bad arguments");
+    return forward_tokens(ctx, m, d_tokens, seqLen, seq, pos, mode, d_logits, d_argmax, 2, nullptr, stream, d_rows, n_rows);
+}
+
+// dst[r] = src[rows[r]]
+__global__ void __launch_bounds__(256) gather_rows_kernel(const float *__restrict__ src, const int *__restrict__ rows, float *__restrict__ dst, int n)
+{
+    smc_grid_dep_sync();
+    for (int i = threadIdx.x; i < n; i += blockDim.x) dst[(size_t)blockIdx.x * n + i] = src[(size_t)rows[blockIdx.x] * n + i];
+}
+
+static int forward_tokens(smc_ctx *ctx, smc_model *m, const int *d_tokens, int seqLen, int seq, int pos, int mode, float *d_logits,
+                          int *d_argmax, int all_rows, float *d_hidden, void *stream, const int *d_rows, int n_rows)
+{
+    if (!ctx || !m || !d_tokens || (!d_logits && all_rows != 2) || seqLen <= 0) return smc_fail(ctx, SMC_E_INVALID, "forward_last_logits: bad arguments");
     if (seq < 0 || seq >= m->max_batch) return smc_fail(ctx, SMC_E_RANGE, "forward_last_logits: sequence %d outside [0, %d)", seq, m->max_batch);
+    if (m->layered) {
+        if (pos < 0) return smc_fail(ctx, SMC_E_RANGE, "forward: position %d", pos);
+        return smc_layered_forward(ctx, m->layered, d_tokens, seqLen, seq, pos, mode, all_rows, d_rows, n_rows, d_logits, d_argmax, d_hidden,
+                                   static_cast<cudaStream_t>(stream));
+    }
     const smc_model_desc &d = m->d;
     if (pos < 0 || (long long)pos + seqLen > d.max_seq)  // KVCache.Update throws on overflow (KVCache.cs:89-91)
         return smc_fail(ctx, SMC_E_RANGE, "KVCache overflow: position %d + seqLen %d exceeds capacity %d", pos, seqLen, d.max_seq);
@@ -643,6 +706,14 @@ static int forward_tokens(smc_ctx *ctx, smc_model *m, const int *d_tokens, int s
         if (d_hidden) SMC_CUDA(ctx, cudaMemcpyAsync(d_hidden, m->xn, (size_t)T * H * sizeof(float), cudaMemcpyDeviceToDevice, s));
         SMC_TRY(smc_qmatmul_dev(ctx, m->xn, d.lm_head, d_logits, T, mode, s));
         if (d_argmax) SMC_TRY(smc_argmax_dev(ctx, d_logits, T, d.vocab, d_argmax, s));
+        return SMC_OK;
+    }
+    if (all_rows == 2) {  // chosen rows
+        if (n_rows == 0) return SMC_OK;
+        smc_launch_dep(ctx->use_pdl, gather_rows_kernel, dim3(n_rows), dim3(256), 0, s, (const float *)m->xn, d_rows, m->x, H);
+        SMC_LAUNCH_CHECK(ctx);
+        SMC_TRY(smc_qmatmul_dev(ctx, m->x, d.lm_head, d_logits, n_rows, mode, s));
+        if (d_argmax) SMC_TRY(smc_argmax_dev(ctx, d_logits, n_rows, d.vocab, d_argmax, s));
         return SMC_OK;
     }
     // only the last position's logits are formed (Transformer.ForwardLastLogits)

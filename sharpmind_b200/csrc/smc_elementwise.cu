@@ -12,6 +12,7 @@
 //   add       SharpMind.Core/Tensors/Tensor.cs:328-332
 //   argmax    SharpMind.Inference/Sampler.cs:50-58
 //   embedding SharpMind.Core/Embeddings/EmbeddingTable.cs:87-116 over ReadQ8_0_Scalar
+#include <cuda_bf16.h>
 #include <math.h>
 
 #include <vector>
@@ -514,6 +515,74 @@ int ew_grid(long long items, int cap)
     return (int)g;
 }
 
+// x = alpha * x + y, then x = x / rms(x) * (w_offset + w): the norm AFTER the residual sum, in place on the fp32 stream,
+// with an optional bfloat16 copy for the matmuls that read it.  A CTA per row; the sum stays in shared memory.
+__global__ void __launch_bounds__(256) scaled_add_rmsnorm_kernel(float *x, const float *__restrict__ y, const float *__restrict__ w,
+                                                                 __nv_bfloat16 *__restrict__ x16, int n, float alpha, float w_offset, float eps)
+{
+    extern __shared__ float row_s[];
+    __shared__ float red[32];
+    smc_grid_dep_sync();
+    float *p = x + (size_t)blockIdx.x * n;
+    const float *q = y ? y + (size_t)blockIdx.x * n : nullptr;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+        const float v = q ? fmaf(alpha, p[i], q[i]) : alpha * p[i];
+        row_s[i] = v;
+        ss = fmaf(v, v, ss);
+    }
+    ss = block_sum(ss, red);
+    const float inv = __fdiv_rn(1.0f, sqrtf(__fdiv_rn(ss, (float)n) + eps));
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+        const float v = (row_s[i] * inv) * (w_offset + w[i]);
+        p[i] = v;
+        if (x16) x16[(size_t)blockIdx.x * n + i] = __float2bfloat16_rn(v);
+    }
+}
+
+// Chosen rows only, into a dense output of either type: out[r] = RMSNorm(x[rows ? rows[r] : first + r]) with w_offset + w.
+__global__ void __launch_bounds__(256) rmsnorm_gather_kernel(const float *__restrict__ x, const int *__restrict__ rows, int first,
+                                                             const float *__restrict__ w, void *out, int out_bf16, int n, float w_offset, float eps)
+{
+    __shared__ float red[32];
+    smc_grid_dep_sync();
+    const float *p = x + (size_t)(rows ? rows[blockIdx.x] : first + (int)blockIdx.x) * n;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < n; i += blockDim.x) ss = fmaf(p[i], p[i], ss);
+    ss = block_sum(ss, red);
+    const float inv = __fdiv_rn(1.0f, sqrtf(__fdiv_rn(ss, (float)n) + eps));
+    for (int i = threadIdx.x; i < n; i += blockDim.x) {
+        const float v = (p[i] * inv) * (w_offset + w[i]);
+        if (out_bf16) static_cast<__nv_bfloat16 *>(out)[(size_t)blockIdx.x * n + i] = __float2bfloat16_rn(v);
+        else static_cast<float *>(out)[(size_t)blockIdx.x * n + i] = v;
+    }
+}
+
+// Rows of a bfloat16 table, widened; the first CTA of a step also moves the sequences on: pos[slot], the position of the
+// step's first row, becomes pos0, or (pos0 < 0) the slot's length, and the length pos[slots + slot] becomes what the
+// slot holds after the step.  A position past the tables raises the status word.
+__global__ void __launch_bounds__(256) embed_bf16_kernel(const __nv_bfloat16 *__restrict__ table, const int *__restrict__ tokens, int H, int vocab,
+                                                         float *__restrict__ out, __nv_bfloat16 *__restrict__ out16, int *pos, int slots, int seq0, int pos0,
+                                                         int max_seq, int *status)
+{
+    smc_grid_dep_sync();
+    const int r = blockIdx.x;
+    if (pos && threadIdx.x == 0 && (seq0 < 0 || r == 0)) {
+        const int slot = seq0 < 0 ? r : seq0;
+        const int p = pos0 >= 0 ? pos0 : pos[slots + slot];
+        pos[slot] = p;
+        pos[slots + slot] = p + (seq0 < 0 ? 1 : (int)gridDim.x);
+        if (p >= max_seq) atomicExch(status, 5);
+    }
+    int tok = tokens[r];
+    tok = tok < 0 ? 0 : (tok >= vocab ? vocab - 1 : tok);
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+        const __nv_bfloat16 v = table[(size_t)tok * H + i];
+        out[(size_t)r * H + i] = __bfloat162float(v);
+        if (out16) out16[(size_t)r * H + i] = v;
+    }
+}
+
 }  // namespace
 
 // Residual add (d_y may be null: none) + RMSNorm with the row leaving as Q8_0 activations in `a`, and as fp32 too when
@@ -744,12 +813,53 @@ int smc_embed_q8_0_dev(smc_ctx *ctx, const smc_weight *table, const int *d_token
     return SMC_OK;
 }
 
+int smc_scaled_add_rmsnorm_dev(smc_ctx *ctx, float *d_x, const float *d_y, const float *d_w, void *d_x16, int rows, int n, float alpha,
+                               float w_offset, float eps, void *stream)
+{
+    if (!ctx || !d_x || !d_w || rows < 0 || n <= 0) return smc_fail(ctx, SMC_E_INVALID, "scaled_add_rmsnorm: bad arguments");
+    const size_t smem = (size_t)n * sizeof(float);
+    if (smem > 200 * 1024) return smc_fail(ctx, SMC_E_UNSUPPORTED, "scaled_add_rmsnorm: rows of %d elements", n);
+    if (rows == 0) return SMC_OK;
+    if (smem > 40 * 1024)
+        SMC_CUDA(ctx, cudaFuncSetAttribute(scaled_add_rmsnorm_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    smc_launch_dep(ctx->use_pdl, scaled_add_rmsnorm_kernel, dim3(rows), dim3(256), smem, static_cast<cudaStream_t>(stream), d_x, d_y, d_w,
+                   static_cast<__nv_bfloat16 *>(d_x16), n, alpha, w_offset, eps);
+    SMC_LAUNCH_CHECK(ctx);
+    return SMC_OK;
+}
+
+int smc_embed_bf16_dev(smc_ctx *ctx, const smc_weight *table, const int *d_tokens, int count, float *d_out, void *stream)
+{
+    if (!ctx || !table || !d_tokens || !d_out || count < 0) return smc_fail(ctx, SMC_E_INVALID, "embed: bad arguments");
+    if (table->dtype != SMC_BF16) return smc_fail(ctx, SMC_E_UNSUPPORTED, "embed: the table is not bfloat16");
+    if (count == 0) return SMC_OK;
+    return smc_launch_embed_bf16(ctx, table, d_tokens, count, d_out, nullptr, nullptr, 0, 0, 0, 1, static_cast<cudaStream_t>(stream));
+}
+
 }  // extern "C"
 
 int smc_launch_rmsnorm_row(smc_ctx *ctx, const float *src, const float *w, float *dst, int n, float rms_inv,
                            cudaStream_t s)
 {
     rmsnorm_row_kernel<<<(n + 255) / 256, 256, 0, s>>>(src, w, dst, n, rms_inv);
+    SMC_LAUNCH_CHECK(ctx);
+    return SMC_OK;
+}
+
+int smc_launch_rmsnorm_gather(smc_ctx *ctx, const float *x, const int *rows, int first, int n_rows, const float *w, void *out, int out_bf16, int n,
+                              float w_offset, float eps, cudaStream_t s)
+{
+    if (n_rows == 0) return SMC_OK;
+    smc_launch_dep(ctx->use_pdl, rmsnorm_gather_kernel, dim3(n_rows), dim3(256), 0, s, x, rows, first, w, out, out_bf16, n, w_offset, eps);
+    SMC_LAUNCH_CHECK(ctx);
+    return SMC_OK;
+}
+
+int smc_launch_embed_bf16(smc_ctx *ctx, const smc_weight *table, const int *tokens, int count, float *x, void *x16, int *pos, int slots, int seq0,
+                          int pos0, int max_seq, cudaStream_t s)
+{
+    smc_launch_dep(ctx->use_pdl, embed_bf16_kernel, dim3(count), dim3(256), 0, s, reinterpret_cast<const __nv_bfloat16 *>(table->d_raw), tokens, table->K,
+                   table->N, x, static_cast<__nv_bfloat16 *>(x16), pos, slots, seq0, pos0, max_seq, ctx->d_status);
     SMC_LAUNCH_CHECK(ctx);
     return SMC_OK;
 }

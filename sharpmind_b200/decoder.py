@@ -29,7 +29,92 @@ class _Desc(C.Structure):
     ]
 
 
-class Decoder:
+class StepModel:
+    """The entry points every model object answers to: one step for a batch of sequences, a pass over several tokens of one
+    sequence, and its cache or state slots.  Subclasses build the handle and set ctx, torch, cfg, max_batch, h and the
+    activation mode they serve with; a call may name another mode."""
+
+    default_mode = ops.Mode.ACT_Q8
+    max_chunk = 2048
+
+    def _mode(self, mode) -> int:
+        return int(self.default_mode if mode is None else mode)
+
+    def step(self, tokens, pos: int, mode: int | None = None, logits=None, argmax=None):
+        """tokens: CUDA int32 [batch]. Returns (logits [batch, vocab], greedy token ids [batch])."""
+        t = self.torch
+        B = tokens.numel()
+        if logits is None:
+            logits = t.empty((B, self.cfg["vocab"]), dtype=t.float32, device="cuda")
+        if argmax is None:
+            argmax = t.empty(B, dtype=t.int32, device="cuda")
+        self.ctx.check(self.ctx.lib.smc_decode_step(self.ctx.h, self.h, tokens.data_ptr(), B, pos, self._mode(mode),
+                                                    logits.data_ptr(), argmax.data_ptr(),
+                                                    C.c_void_p(t.cuda.current_stream().cuda_stream)))
+        return logits, argmax
+
+    def forward_last_logits(self, tokens, pos: int = 0, seq: int = 0, mode: int | None = None, chunk: int | None = None):
+        """Prompt processing (Transformer.ForwardLastLogits with seqLen > 1): tokens is CUDA int32 [seqLen], one
+        sequence, placed at positions pos .. pos + seqLen - 1 of cache slot `seq`, fed in chunks of `chunk` tokens.
+        Returns (logits [vocab] of the last token, its greedy pick [1])."""
+        t = self.torch
+        n, chunk = tokens.numel(), chunk or self.max_chunk
+        logits = t.empty(self.cfg["vocab"], dtype=t.float32, device="cuda")
+        argmax = t.empty(1, dtype=t.int32, device="cuda")
+        if n == 0:
+            raise ValueError("forward_last_logits: empty prompt")
+        for start in range(0, n, chunk):
+            part = tokens[start:start + chunk].contiguous()
+            self.ctx.check(self.ctx.lib.smc_forward_last_logits(self.ctx.h, self.h, part.data_ptr(), part.numel(), seq,
+                                                                pos + start, self._mode(mode), logits.data_ptr(), argmax.data_ptr(),
+                                                                C.c_void_p(t.cuda.current_stream().cuda_stream)))
+        return logits, argmax
+
+    def forward_logits(self, tokens, pos: int, seq: int = 0, mode: int | None = None, want_hidden: bool = False):
+        """Transformer.Forward over the tokens of one sequence (a verification round's K + 1 draft tokens): returns
+        (logits [seqLen, vocab], greedy pick per row [seqLen], final-normed hidden states [seqLen, hidden] or None)."""
+        t = self.torch
+        n = tokens.numel()
+        logits = t.empty((n, self.cfg["vocab"]), dtype=t.float32, device="cuda")
+        argmax = t.empty(n, dtype=t.int32, device="cuda")
+        hidden = t.empty((n, self.cfg["hidden"]), dtype=t.float32, device="cuda") if want_hidden else None
+        self.ctx.check(self.ctx.lib.smc_forward_logits(self.ctx.h, self.h, tokens.contiguous().data_ptr(), n, seq, pos, self._mode(mode),
+                                                       logits.data_ptr(), argmax.data_ptr(),
+                                                       None if hidden is None else hidden.data_ptr(),
+                                                       C.c_void_p(t.cuda.current_stream().cuda_stream)))
+        return logits, argmax, hidden
+
+    def forward_rows(self, tokens, pos: int, seq: int = 0, rows=None, mode: int | None = None, argmax=None):
+        """A portion of one sequence (up to max_chunk tokens) of which only the places `rows` (CUDA int32, may be None)
+        meet the LM head: logits [len(rows), vocab], or None."""
+        t = self.torch
+        n = 0 if rows is None else rows.numel()
+        logits = t.empty((n, self.cfg["vocab"]), dtype=t.float32, device="cuda") if n else None
+        self.ctx.check(self.ctx.lib.smc_forward_rows(self.ctx.h, self.h, tokens.contiguous().data_ptr(), tokens.numel(), seq, pos, self._mode(mode),
+                                                     rows.data_ptr() if n else None, n, logits.data_ptr() if n else None,
+                                                     None if argmax is None else argmax.data_ptr(),
+                                                     C.c_void_p(t.cuda.current_stream().cuda_stream)))
+        return logits
+
+    def reset_sequence(self, seq: int):
+        """Forgets what slot `seq` holds: it may start another sequence."""
+        self.ctx.check(self.ctx.lib.smc_model_seq_reset(self.ctx.h, self.h, seq))
+
+    def verify_greedy(self, argmax, draft):
+        """1 + the number of leading head guesses the model agrees with (MedusaGenerator's acceptance rule)."""
+        t = self.torch
+        acc = t.zeros(1, dtype=t.int32, device="cuda")
+        self.ctx.check(self.ctx.lib.smc_verify_greedy_dev(self.ctx.h, argmax.data_ptr(), draft.contiguous().data_ptr(), draft.numel() - 1,
+                                                          acc.data_ptr(), C.c_void_p(t.cuda.current_stream().cuda_stream)))
+        return int(acc.item())
+
+    def close(self):
+        if self.h:
+            self.ctx.lib.smc_model_destroy(self.ctx.h, self.h)
+            self.h = None
+
+
+class Decoder(StepModel):
     def __init__(self, ctx: ops.CudaContext, cfg: dict, weights: dict, max_batch: int, keep_raw: bool = False):
         import torch
 
@@ -109,58 +194,6 @@ class Decoder:
                                                       v.contiguous().data_ptr(), B, ln,
                                                       C.c_void_p(self.torch.cuda.current_stream().cuda_stream)))
 
-    def step(self, tokens, pos: int, mode: int = ops.Mode.ACT_Q8, logits=None, argmax=None):
-        """tokens: CUDA int32 [batch]. Returns (logits [batch, vocab], greedy token ids [batch])."""
-        t = self.torch
-        B = tokens.numel()
-        if logits is None:
-            logits = t.empty((B, self.cfg["vocab"]), dtype=t.float32, device="cuda")
-        if argmax is None:
-            argmax = t.empty(B, dtype=t.int32, device="cuda")
-        self.ctx.check(self.ctx.lib.smc_decode_step(self.ctx.h, self.h, tokens.data_ptr(), B, pos, int(mode),
-                                                    logits.data_ptr(), argmax.data_ptr(),
-                                                    C.c_void_p(t.cuda.current_stream().cuda_stream)))
-        return logits, argmax
-
-    def forward_last_logits(self, tokens, pos: int = 0, seq: int = 0, mode: int = ops.Mode.ACT_Q8, chunk: int = 2048):
-        """Prompt processing (Transformer.ForwardLastLogits with seqLen > 1): tokens is CUDA int32 [seqLen], one
-        sequence, placed at positions pos .. pos + seqLen - 1 of cache slot `seq`, fed in chunks of `chunk` tokens.
-        Returns (logits [vocab] of the last token, its greedy pick [1])."""
-        t = self.torch
-        n = tokens.numel()
-        logits = t.empty(self.cfg["vocab"], dtype=t.float32, device="cuda")
-        argmax = t.empty(1, dtype=t.int32, device="cuda")
-        if n == 0:
-            raise ValueError("forward_last_logits: empty prompt")
-        for start in range(0, n, chunk):
-            part = tokens[start:start + chunk].contiguous()
-            self.ctx.check(self.ctx.lib.smc_forward_last_logits(self.ctx.h, self.h, part.data_ptr(), part.numel(), seq,
-                                                                pos + start, int(mode), logits.data_ptr(), argmax.data_ptr(),
-                                                                C.c_void_p(t.cuda.current_stream().cuda_stream)))
-        return logits, argmax
-
-    def forward_logits(self, tokens, pos: int, seq: int = 0, mode: int = ops.Mode.ACT_Q8, want_hidden: bool = False):
-        """Transformer.Forward over the tokens of one sequence (a verification round's K + 1 draft tokens): returns
-        (logits [seqLen, vocab], greedy pick per row [seqLen], final-normed hidden states [seqLen, hidden] or None)."""
-        t = self.torch
-        n = tokens.numel()
-        logits = t.empty((n, self.cfg["vocab"]), dtype=t.float32, device="cuda")
-        argmax = t.empty(n, dtype=t.int32, device="cuda")
-        hidden = t.empty((n, self.cfg["hidden"]), dtype=t.float32, device="cuda") if want_hidden else None
-        self.ctx.check(self.ctx.lib.smc_forward_logits(self.ctx.h, self.h, tokens.contiguous().data_ptr(), n, seq, pos, int(mode),
-                                                       logits.data_ptr(), argmax.data_ptr(),
-                                                       None if hidden is None else hidden.data_ptr(),
-                                                       C.c_void_p(t.cuda.current_stream().cuda_stream)))
-        return logits, argmax, hidden
-
-    def verify_greedy(self, argmax, draft):
-        """1 + the number of leading head guesses the model agrees with (MedusaGenerator's acceptance rule)."""
-        t = self.torch
-        acc = t.zeros(1, dtype=t.int32, device="cuda")
-        self.ctx.check(self.ctx.lib.smc_verify_greedy_dev(self.ctx.h, argmax.data_ptr(), draft.contiguous().data_ptr(), draft.numel() - 1,
-                                                          acc.data_ptr(), C.c_void_p(t.cuda.current_stream().cuda_stream)))
-        return int(acc.item())
-
     def medusa_predict(self, hidden, head_w, head_b):
         """MedusaHeads.Predict: hidden [hidden] (final-normed), head_w [k, hidden, hidden], head_b [k, hidden] -> tokens [k]."""
         t = self.torch
@@ -171,8 +204,3 @@ class Decoder:
                                                            head_b.contiguous().data_ptr(), k, H, self.embedding.handle, work.data_ptr(),
                                                            out.data_ptr(), C.c_void_p(t.cuda.current_stream().cuda_stream)))
         return out
-
-    def close(self):
-        if self.h:
-            self.ctx.lib.smc_model_destroy(self.ctx.h, self.h)
-            self.h = None

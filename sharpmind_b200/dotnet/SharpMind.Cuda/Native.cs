@@ -154,6 +154,19 @@ internal static unsafe partial class Native
     [LibraryImport(Lib)] internal static partial int smc_medusa_predict_dev(nint ctx, nint dHidden, nint dHeadW, nint dHeadB, int k, int hidden,
         nint lmHead, nint dWork, nint dTokens, nint stream);
 
+    [LibraryImport(Lib)] internal static partial int smc_forward_rows(nint ctx, nint model, nint dTokens, int seqLen, int seq, int pos,
+        int mode, nint dRows, int nRows, nint dLogits, nint dArgmax, nint stream);
+
+    // ---- layered decoders (desc: a smc_layered_desc laid out in unmanaged memory)
+    [LibraryImport(Lib)] internal static partial int smc_model_create_layered(nint ctx, nint desc, int maxBatch, out nint model);
+    [LibraryImport(Lib)] internal static partial int smc_model_seq_length(nint ctx, nint model, int seq, out int length);
+    [LibraryImport(Lib)] internal static partial int smc_model_seq_reset(nint ctx, nint model, int seq);
+    [LibraryImport(Lib)] internal static partial int smc_model_dump_layers(nint ctx, nint model, nint dDump);
+    [LibraryImport(Lib)] internal static partial int smc_rope_tables_yarn(nint ctx, nint rotation, int maxSeq, nint dCos, nint dSin);
+    [LibraryImport(Lib)] internal static partial int smc_scaled_add_rmsnorm_dev(nint ctx, nint dX, nint dY, nint dW, nint dX16, int rows, int n,
+        float alpha, float wOffset, float eps, nint stream);
+    [LibraryImport(Lib)] internal static partial int smc_embed_bf16_dev(nint ctx, nint table, nint dTokens, int count, nint dOut, nint stream);
+
     // ---- GGUF
     [LibraryImport(Lib, StringMarshalling = StringMarshalling.Utf8)]
     internal static partial int smc_gguf_open(nint ctx, string path, out nint gguf);

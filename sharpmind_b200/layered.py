@@ -1,0 +1,194 @@
+"""Decoders described layer by layer: configuration, weight loading and the device model (smc_model_create_layered).
+
+A configuration names for every layer its sequence mixer ('latent_attention' or 'mamba2'), the mixer's sizes and its
+feed-forward; `read_config` turns the JSON form into the plain description `LayeredDecoder` takes.  Matrices stay bfloat16
+on the device; projections that read the same rows are joined (smc_weight_concat_rows), gate and up rows are woven
+(smc_weight_interleave_rows).  A layer with 'weights_of' shares another layer's handles and has a state of its own.
+"""
+from __future__ import annotations
+
+import ctypes as C
+
+from . import ops
+from .decoder import StepModel
+
+MIX_LATENT, MIX_MAMBA2 = 1, 2
+POS_NEXT = -1  # StepModel.step: every slot's next position, taken from the device
+
+
+class _Rotation(C.Structure):
+    _fields_ = [("dims", C.c_int), ("base", C.c_double), ("factor", C.c_double), ("original", C.c_double), ("fast", C.c_double),
+                ("slow", C.c_double)]
+
+
+class _Layer(C.Structure):
+    _fields_ = [
+        ("mixer", C.c_int), ("heads", C.c_int), ("vdim", C.c_int),
+        ("dim", C.c_int), ("rot_dim", C.c_int), ("q_rank", C.c_int), ("kv_rank", C.c_int), ("window", C.c_int),
+        ("scale", C.c_float), ("rot", _Rotation), ("w_down", C.c_void_p), ("w_uq", C.c_void_p), ("w_ukv", C.c_void_p),
+        ("q_norm", C.c_void_p), ("kv_norm", C.c_void_p), ("sink", C.c_void_p),
+        ("state", C.c_int), ("groups", C.c_int), ("conv", C.c_int), ("norm_groups", C.c_int), ("w_in", C.c_void_p),
+        ("conv_w", C.c_void_p), ("conv_b", C.c_void_p), ("dt_bias", C.c_void_p), ("a_log", C.c_void_p), ("d_skip", C.c_void_p),
+        ("mix_norm", C.c_void_p), ("w_out", C.c_void_p),
+        ("ffn", C.c_int), ("w_gu", C.c_void_p), ("w_ffn_down", C.c_void_p), ("norm1", C.c_void_p), ("norm2", C.c_void_p),
+    ]
+
+
+class _Desc(C.Structure):
+    _fields_ = [
+        ("n_layers", C.c_int), ("hidden", C.c_int), ("vocab", C.c_int), ("max_seq", C.c_int), ("max_chunk", C.c_int),
+        ("act_dtype", C.c_int), ("eps", C.c_float), ("alpha", C.c_float), ("layers", C.POINTER(_Layer)), ("embedding", C.c_void_p),
+        ("final_norm", C.c_void_p),
+    ]
+
+
+def rotation(rot: dict) -> _Rotation:
+    s = rot.get("scaling") or {}
+    return _Rotation(int(rot["dims"]), float(rot["base"]), float(s.get("factor", 0.0)), float(s.get("original", 0.0)),
+                     float(s.get("fast", 0.0)), float(s.get("slow", 0.0)))
+
+
+def read_config(raw: dict) -> dict:
+    """The JSON configuration of a layered decoder, checked: {"vocab", "hidden", "eps", "alpha", "layers": [...]}."""
+    layers = []
+    for i, e in enumerate(raw["layers"]):
+        kind, src = e["type"], e.get("weights_of", i)
+        if kind not in ("latent_attention", "mamba2"):
+            raise ops.NotSupportedException(f"layer {i}: mixer '{kind}'")
+        mlp = e.get("mlp")
+        if mlp and mlp.get("kind", "dense") != "dense":
+            raise ops.NotSupportedException(f"layer {i}: feed-forward '{mlp['kind']}'")
+        if not 0 <= src < len(raw["layers"]) or "weights_of" in raw["layers"][src]:
+            raise ops.ArgumentException(f"layer {i}: weights of layer {src}")
+        if src != i and raw["layers"][src]["type"] != kind:
+            raise ops.ArgumentException(f"layer {i} ({kind}) cannot use the weights of layer {src} ({raw['layers'][src]['type']})")
+        layers.append({"type": kind, "weights_of": src, "mixer": dict(e["mixer"]), "ffn": int(mlp["ff"]) if mlp else 0})
+    return {"vocab": int(raw["vocab"]), "hidden": int(raw["width"]), "eps": float(raw["norm"]["eps"]), "alpha": float(raw["postln_alpha"]),
+            "layers": layers}
+
+
+def tensor_shapes(cfg: dict) -> dict:
+    """Name -> shape of every tensor of a configuration."""
+    H = cfg["hidden"]
+    out = {"embed": (cfg["vocab"], H), "final.norm": (H,)}
+    for i, L in enumerate(cfg["layers"]):
+        if L["weights_of"] != i:
+            continue
+        p, m = f"l{i}.", L["mixer"]
+        out[p + "norm1"] = (H,)
+        if L["type"] == "latent_attention":
+            h, dn, dr, dv, qr, rk = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["q_rank"], m["kv_rank"]
+            out.update({p + "mix.dq": (qr, H), p + "mix.dq.norm": (qr,), p + "mix.uq": (h * (dn + dr), qr), p + "mix.dkv": (rk + dr, H),
+                        p + "mix.dkv.norm": (rk,), p + "mix.uk": (h * dn, rk), p + "mix.uv": (h * dv, rk), p + "mix.sink": (h,),
+                        p + "mix.o": (H, h * dv)})
+        else:
+            h, inner, bc = m["heads"], m["heads"] * m["vdim"], m["groups"] * m["state"]
+            ch = inner + 2 * bc
+            out.update({p + "mix.in": (inner + ch + h, H), p + "mix.conv": (ch, m["conv"]), p + "mix.conv.b": (ch,), p + "mix.dt_bias": (h,),
+                        p + "mix.A_log": (h,), p + "mix.D": (h,), p + "mix.norm": (inner,), p + "mix.o": (H, inner)})
+        if L["ffn"]:
+            out.update({p + "norm2": (H,), p + "mlp.gate": (L["ffn"], H), p + "mlp.up": (L["ffn"], H), p + "mlp.down": (H, L["ffn"])})
+    return out
+
+
+class LayeredDecoder(StepModel):
+    """`tensors`: a mapping from tensor name to a torch tensor (CPU or CUDA), matrices in bfloat16.  `act`: "bfloat16"
+    (activations and latent cache in bfloat16, the serving form) or "float32" (everything in fp32)."""
+
+    def __init__(self, ctx: ops.CudaContext, cfg: dict, tensors, max_batch: int, max_seq: int, max_chunk: int = 2048, act: str = "bfloat16"):
+        import torch
+
+        self.torch, self.ctx, self.max_batch = torch, ctx, max_batch
+        self.cfg = dict(cfg, max_seq=max_seq)
+        self.act = act
+        self.default_mode = {"bfloat16": ops.Mode.ACT_BF16, "float32": ops.Mode.ACT_F32}[act]
+        self.max_chunk = min(max_chunk, max_seq)
+        self._keep, self.weights = [], []
+        self._dev = ops.DeviceOps(ctx)
+        self.h = None
+        shapes = tensor_shapes(cfg)
+
+        def fetch(name):
+            t = tensors[name]
+            if tuple(t.shape) != tuple(shapes[name]):
+                raise ops.InvalidOperationException(f"tensor '{name}' is {tuple(t.shape)}, the configuration needs {shapes[name]}")
+            return t
+
+        def mat(name):
+            t = fetch(name)
+            if t.dtype != torch.bfloat16:
+                raise ops.NotSupportedException(f"tensor '{name}' is {t.dtype}; matrices are bfloat16")
+            t = t.contiguous().cuda()
+            return ctx.register_dev(t.view(torch.uint8).reshape(-1), ops.QuantDType.BF16, t.shape[0], t.shape[1], repack=False)
+
+        def own(w):
+            self.weights.append(w)
+            return w.handle
+
+        def joined(*names):
+            parts = [mat(n) for n in names]
+            w = ctx.concat_rows(parts)
+            for p in parts:
+                ctx.release(p)
+            return own(w)
+
+        def woven(gate, up):
+            a, b = mat(gate), mat(up)
+            w = self._dev.interleave_rows(a, b)
+            ctx.release(a), ctx.release(b)
+            return own(w)
+
+        def vec(name):
+            t = fetch(name).to(torch.float32).contiguous().cuda()
+            self._keep.append(t)
+            return t.data_ptr()
+
+        descs = (_Layer * len(cfg["layers"]))()
+        for i, L in enumerate(cfg["layers"]):
+            d, m, p = descs[i], L["mixer"], f"l{L['weights_of']}."
+            if L["weights_of"] != i:
+                continue
+            d.heads, d.vdim, d.ffn = m["heads"], m["vdim"], L["ffn"]
+            d.norm1, d.w_out = vec(p + "norm1"), own(mat(p + "mix.o"))
+            if L["type"] == "latent_attention":
+                d.mixer = MIX_LATENT
+                d.dim, d.rot_dim, d.q_rank, d.kv_rank = m["dim"], m["rot_dim"], m["q_rank"], m["kv_rank"]
+                d.window, d.scale, d.rot = int((m.get("mask") or {}).get("size", 0)), m["scale"], rotation(m["rot"])
+                d.w_down, d.w_uq = joined(p + "mix.dq", p + "mix.dkv"), own(mat(p + "mix.uq"))
+                d.w_ukv = joined(p + "mix.uk", p + "mix.uv")
+                d.q_norm, d.kv_norm, d.sink = vec(p + "mix.dq.norm"), vec(p + "mix.dkv.norm"), vec(p + "mix.sink")
+            else:
+                d.mixer = MIX_MAMBA2
+                d.state, d.groups, d.conv, d.norm_groups = m["state"], m["groups"], m["conv"], m["norm_groups"]
+                d.w_in = own(mat(p + "mix.in"))
+                d.conv_w, d.conv_b, d.dt_bias = vec(p + "mix.conv"), vec(p + "mix.conv.b"), vec(p + "mix.dt_bias")
+                d.a_log, d.d_skip, d.mix_norm = vec(p + "mix.A_log"), vec(p + "mix.D"), vec(p + "mix.norm")
+            if L["ffn"]:
+                d.w_gu, d.w_ffn_down, d.norm2 = woven(p + "mlp.gate", p + "mlp.up"), own(mat(p + "mlp.down")), vec(p + "norm2")
+        for i, L in enumerate(cfg["layers"]):
+            if L["weights_of"] != i:
+                C.memmove(C.byref(descs[i]), C.byref(descs[L["weights_of"]]), C.sizeof(_Layer))
+        desc = _Desc(len(cfg["layers"]), cfg["hidden"], cfg["vocab"], max_seq, max_chunk,
+                     int(ops.QuantDType.BF16) if act == "bfloat16" else 0, cfg["eps"], cfg["alpha"], descs, own(mat("embed")), vec("final.norm"))
+        h = C.c_void_p()
+        torch.cuda.synchronize()
+        ctx.check(ctx.lib.smc_model_create_layered(ctx.h, C.byref(desc), max_batch, C.byref(h)))
+        self.h = h
+
+    def sequence_length(self, seq: int) -> int:
+        n = C.c_int()
+        self.ctx.check(self.ctx.lib.smc_model_seq_length(self.ctx.h, self.h, seq, C.byref(n)))
+        return n.value
+
+    def dump_layers(self, on: bool = True):
+        """The residual stream after every layer of the following passes: [n_layers, max_chunk, hidden] (None to stop)."""
+        t = self.torch
+        self._dump = t.zeros((len(self.cfg["layers"]), self.max_chunk, self.cfg["hidden"]), device="cuda") if on else None
+        self.ctx.check(self.ctx.lib.smc_model_dump_layers(self.ctx.h, self.h, self._dump.data_ptr() if on else None))
+        return self._dump
+
+    def close(self):
+        super().close()
+        for w in self.weights:
+            self.ctx.release(w)
+        self.weights = []

@@ -47,12 +47,14 @@ class QuantDType(IntEnum):  # SharpMind.Core/Quantization/QuantDType.cs:2-18
     Q8_0 = 8
     Q4_K = 12
     Q6_K = 14
+    BF16 = 30  # dense; GGUF's number for it
 
 
 class Mode(IntEnum):
     ACT_F32 = 0
     ACT_Q8 = 1
     REF_ORDER = 2
+    ACT_BF16 = 3
 
 
 W_REPACK, W_KEEP_RAW = 1, 2
@@ -147,6 +149,13 @@ class CudaContext:
         self.check(self.lib.smc_weight_register_dev(self.h, raw.data_ptr(), raw.numel(), int(dtype), n, k, flags,
                                                     C.byref(h)))
         return Weight(h, dtype, n, k, None)
+
+    def concat_rows(self, parts: list[Weight]) -> Weight:
+        """One weight whose rows are the parts' rows in order (smc_weight_concat_rows)."""
+        h = C.c_void_p()
+        hs = (C.c_void_p * len(parts))(*[p.handle for p in parts])
+        self.check(self.lib.smc_weight_concat_rows(self.h, hs, len(parts), C.byref(h)))
+        return Weight(h, parts[0].dtype, sum(p.N for p in parts), parts[0].K, None)
 
     def lookup(self, raw: np.ndarray) -> C.c_void_p:
         h = C.c_void_p()
@@ -539,6 +548,23 @@ class DeviceOps:
         self.ctx.check(self.lib.smc_embed_q8_0_dev(self.ctx.h, table.handle, self._chk(tokens, t.int32), tokens.numel(),
                                                    self._chk(out), self._stream()))
         return out
+
+    def embed_bf16(self, table: Weight, tokens, out=None):
+        t = self.torch
+        if out is None:
+            out = t.empty((tokens.numel(), table.K), dtype=t.float32, device=tokens.device)
+        self.ctx.check(self.lib.smc_embed_bf16_dev(self.ctx.h, table.handle, self._chk(tokens, t.int32), tokens.numel(),
+                                                   self._chk(out), self._stream()))
+        return out
+
+    def scaled_add_rmsnorm_(self, x, y, w, alpha: float, eps: float, w_offset: float = 1.0, x16=None):
+        """x = norm(alpha * x + y) * (w_offset + w) in place (y may be None); `x16` also receives the rows in bfloat16."""
+        rows, n = x.shape
+        self.ctx.check(self.lib.smc_scaled_add_rmsnorm_dev(
+            self.ctx.h, self._chk(x, self.torch.float32), None if y is None else self._chk(y, self.torch.float32),
+            self._chk(w, self.torch.float32), None if x16 is None else self._chk(x16, self.torch.bfloat16), rows, n, C.c_float(alpha),
+            C.c_float(w_offset), C.c_float(eps), self._stream()))
+        return x
 
     def sdpa_decode(self, q, kcache, vcache, kv_len: int, scale: float, out=None):
         """q [batch, heads, hd]; caches [batch, kv_heads, max_seq, hd]."""
