@@ -2,7 +2,8 @@
 
     python bench.py [--gpus N] [--steps K] [--warmup W] [--impl ours|reference]
                     [--workload llama70b|llama8b] [--batch M] [--mode q8|f32] [--layers L]
-                    [--only gemv:<shape>[:<M>[:q8|q8pre|f32[:ring]]] | decode[:qwen3|llama8b][:q8kv] | prompt[:llama8b] | elementwise | prefill]
+                    [--only gemv:<shape>[:<M>[:q8|q8pre|f32[:ring]]] | decode[:qwen3|llama8b][:q8kv] | prompt[:llama8b] | elementwise | prefill
+                            | layered[:<size>][:prompt|decode|ours]]
 
 Workload (default `llama70b`, BASELINE configs[4], the largest configuration that fits one GPU and the one the
 multi-GPU target is stated on): the Llama-3-70B-shaped FFN GEMV stack -- per layer the fused gate||up projection
@@ -31,6 +32,10 @@ along K and its partial sums are exchanged and added in rank order inside the GE
 `--tp rows` splits every matrix by rows and exchanges the output slices of every matmul inside the kernel;
 `--gather nccl` uses a library all-gather per matmul instead.  Total work is fixed ("strong" scaling).
 `--impl reference` times the CPU port alone on a bounded sample per step (rank 0 only, all host threads).
+`--only layered` times the layered decoder (alternating latent attention and Mamba-2 layers, bfloat16) at the sizes of
+LAYERED_SIZES beside the Llama-shaped decoder (Q8_0) of the same width, depth, feed-forward and vocabulary: a 2048-token
+prompt and decode steps at batch 1 and 32; `:decode` / `:prompt` runs one pass of one size without a graph (the form a
+launch list wants), `:ours` leaves the other model out.
 `--only ...` runs one kernel or section by itself and prints its own JSON line: the commands behind profiles/.
 """
 from __future__ import annotations
@@ -70,6 +75,16 @@ GEMV_SHAPES = {
 # algorithmic bytes, the rest are dirty lines of earlier kernels leaving the L2 during the capture); traffic grows with
 # the rows a launch covers, so other shapes scale it.
 NCU_TRAFFIC_PER_ALGORITHMIC_BYTE = {Q4_K: 1.022, Q6_K: 1.044, Q8_0: 1.040}
+
+
+# --only layered:<size>: layer sizes that resemble real models', (hidden, layers, ffn, vocab, attention heads, latent ranks
+# (q, kv), window, state-space heads); per head 128 unrotated + 64 rotated query/key and 128 value elements, states of
+# 128 x 64 in 8 groups, four convolution taps
+LAYERED_SIZES = {
+    "w1024": (1024, 16, 3072, 32000, 8, 384, 256, 1024, 32),
+    "w2048": (2048, 16, 5632, 32000, 16, 768, 512, 1024, 64),
+    "w4096": (4096, 8, 14336, 32000, 32, 1536, 512, 4096, 128),
+}
 
 
 def parse():
@@ -505,6 +520,108 @@ def prefill_section(torch, ctx, dev, ops, peaks: dict, n: int, k: int, layers: i
             "peak_source": "measured bf16 burst (MEASURED_PEAKS.json)" if "bf16_tflops" in peaks else "fallback"}
 
 
+def layered_config(size: str) -> dict:
+    """A configuration of LAYERED_SIZES in the form layered.read_config returns: latent attention and Mamba-2 in turn."""
+    H, L, F, V, heads, qr, kr, window, sh = LAYERED_SIZES[size]
+    rot = {"base": 500000.0, "dims": 64, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}
+    lat = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": qr, "kv_rank": kr, "mask": {"size": window}, "scale": 192 ** -0.5, "rot": rot}
+    ssm = {"heads": sh, "vdim": 64, "state": 128, "groups": 8, "conv": 4, "norm_groups": 8}
+    layers = [{"type": ("latent_attention", "mamba2")[i & 1], "weights_of": i, "mixer": (lat, ssm)[i & 1], "ffn": F} for i in range(L)]
+    return {"vocab": V, "hidden": H, "eps": 1e-5, "alpha": (2 * L) ** 0.25, "layers": layers}
+
+
+class LayeredDeviceWeights:
+    """Random bfloat16 tensors of a configuration, drawn on the device when asked for."""
+
+    def __init__(self, torch, cfg: dict):
+        from sharpmind_b200 import layered
+
+        self.torch, self.shapes = torch, layered.tensor_shapes(cfg)
+        self.g = torch.Generator(device="cuda").manual_seed(4321)
+
+    def __getitem__(self, name: str):
+        t, shape, last = self.torch, self.shapes[name], name.split(".", 1)[-1]
+        x = t.randn(shape, generator=self.g, device="cuda")
+        if last == "mix.A_log":
+            x = x * 0.5
+        elif last == "mix.dt_bias":
+            x = x * 0.5 - 2.0
+        elif last in ("mix.dq.norm", "mix.dkv.norm", "mix.norm"):
+            x = 1.0 + 0.1 * x
+        elif len(shape) == 1:
+            x = 0.1 * x
+        elif last != "mix.conv":
+            x = x * shape[1] ** -0.5
+        return x.to(t.bfloat16)
+
+
+def layered_section(torch, ctx, dev, size: str, batches, steps: int, n_prompt: int, once: str = "", ours_only: bool = False) -> dict:
+    """Prompt and decode throughput of the layered decoder, and of the Llama-shaped Q8_0 decoder of equal size."""
+    from sharpmind_b200 import layered, ops
+
+    cfg = layered_config(size)
+    H, L, F, V, heads = LAYERED_SIZES[size][:5]
+    weights = LayeredDeviceWeights(torch, cfg)
+    max_seq = n_prompt + 4 * steps + 64
+    m = layered.LayeredDecoder(ctx, cfg, weights, max_batch=max(batches), max_seq=max_seq, max_chunk=n_prompt)
+    params = sum(int(np.prod(sh)) for sh in weights.shapes.values())
+    g = torch.Generator(device="cuda").manual_seed(7)
+    tok = torch.randint(0, V, (n_prompt,), generator=g, device="cuda", dtype=torch.int32)
+    row = {"size": size, "hidden": H, "layers": L, "ffn": F, "vocab": V, "parameters_M": round(params / 1e6, 1)}
+
+    def rewind(b):
+        for i in range(b):
+            m.reset_sequence(i)
+
+    if once == "prompt":
+        m.forward_last_logits(tok, 0, 0)
+        torch.cuda.synchronize()
+        return row
+    if once == "decode":
+        for b in batches:
+            t1 = tok[:b].contiguous()
+            m.step(t1, 0)
+            m.step(t1, layered.POS_NEXT)
+        torch.cuda.synchronize()
+        return row
+
+    def prompt_ms(fn, reps=5):
+        for _ in range(2):
+            fn()
+        torch.cuda.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        for _ in range(reps):
+            fn()
+        e1.record()
+        torch.cuda.synchronize()
+        return e0.elapsed_time(e1) / reps
+
+    ms = prompt_ms(lambda: m.forward_last_logits(tok, 0, 0))
+    row["prompt"] = {"tokens": n_prompt, "ms": round(ms, 3), "tokens_per_s": round(n_prompt / ms * 1e3, 1)}
+    row["decode"] = []
+    for b in batches:
+        for i in range(b):  # every sequence holds its own prompt
+            m.forward_rows(tok.roll(i), 0, i)
+        t1 = tok[:b].contiguous()
+        logits, nxt = torch.empty((b, V), device="cuda"), torch.empty(b, dtype=torch.int32, device="cuda")
+        us = time_graph_us(torch, lambda: m.step(t1, layered.POS_NEXT, logits=logits, argmax=nxt), 1, reps=steps)
+        row["decode"].append({"batch": b, "ctx": n_prompt, "ms_per_step": round(us / 1e3, 4), "tokens_per_s": round(b / us * 1e6, 1),
+                              "weight_GBps": round(2 * params / us / 1e3, 1)})
+        rewind(b)
+    row["device_status"] = ctx.device_status()
+    m.close()
+    if not ours_only:
+        # Llama-shaped, every matrix Q8_0, head size 128, grouped KV heads
+        like = dict(n_layers=L, hidden=H, n_heads=H // 128, n_kv_heads=max(1, H // 256), head_dim=128, ffn=F, vocab=V, max_seq=n_prompt + 64, dtype=8,
+                    eps=1e-5, rope_theta=5.0e5, neox=False, qk_norm=False)
+        p = time_prompt(torch, ctx, dev, like, n_prompt, n_prompt, ops.Mode.ACT_Q8)
+        d = time_decode(torch, ctx, dev, like, list(batches), n_prompt, steps, ops.Mode.ACT_Q8)
+        row["llama_shaped_q8_0"] = {"prompt": {k: p[k] for k in ("ms", "tokens_per_s")},
+                                    "decode": [{k: x[k] for k in ("batch", "ms_per_step", "tokens_per_s", "weight_MB", "kv_MB")} for x in d]}
+    return row
+
+
 def run_only(args):
     import torch
 
@@ -538,6 +655,11 @@ def run_only(args):
         res = {"elementwise": elementwise_chain(torch, ctx, dev, peak, once=args.no_graph)}
     elif parts[0] == "prefill":
         res = {"prefill": prefill_section(torch, ctx, dev, ops, peaks, 28672, 8192, 2)}
+    elif parts[0] == "layered":
+        sizes = [p for p in parts[1:] if p in LAYERED_SIZES] or list(LAYERED_SIZES)
+        once = next((p for p in parts[1:] if p in ("prompt", "decode")), "")
+        batches = [args.batch] if once else [1, 32]
+        res = {"layered": [layered_section(torch, ctx, dev, sz, batches, max(args.steps, 4), 2048, once, "ours" in parts) for sz in sizes]}
     else:
         raise SystemExit(f"unknown --only section '{args.only}'")
     print(json.dumps(res), flush=True)

@@ -208,6 +208,10 @@ int smc_launch_dense(smc_ctx *, const void *x, int x_bf16, int ldx, const smc_we
 int smc_launch_dense_rows(smc_ctx *, const void *x, int x_bf16, int ldx, const smc_weight *, int row0, int N, int M, const smc_dense_out &,
                           cudaStream_t s);
 int smc_launch_round_bf16(smc_ctx *, const float *x, void *y, long long n, cudaStream_t s);
+// few bfloat16 rows against `groups` stacked matrices [N, K]: group z reads columns z * x_group .. + K - 1 of x and makes
+// columns z * N .. of the product
+int smc_launch_dense_grouped(smc_ctx *, const void *x, int ldx, int x_group, const void *w, int groups, int N, int K, int M, const smc_dense_out &,
+                             cudaStream_t s);
 // Row r of a batch: of sequence slot seq0 at position pos[seq0] + r, or (seq0 < 0) of slot r at position pos[r].
 struct smc_rows {
     const int *pos;
@@ -230,7 +234,8 @@ struct smc_latent_bufs {          // activation buffers of a step, element type 
     void *cq;                     // [rows, q_rank]  T
     const void *q;                // [rows, heads * (dim + rot_dim)]  T
     float *qa;                    // [rows, heads, kv_rank + rot_dim]
-    float *oc;                    // [rows, heads, kv_rank]
+    void *oc;                     // [rows, heads, kv_rank]  fp32 (bfloat16 between the tensor-core kernels)
+    const void *w_ukt;            // [heads, kv_rank, dim] bfloat16: every head's key expansion transposed (may be null)
     void *o;                      // [rows, heads * vdim]  T
     void *keys;                   // [window - 1 + rows, kv_rank + rot_dim]  T
     void *kv;                     // [window - 1 + rows, heads * (dim + vdim)]  T
@@ -240,8 +245,10 @@ int smc_latent_post(smc_ctx *, const smc_latent_dims &, const smc_latent_bufs &,
                     const float *kv_norm, const float *cosT, const float *sinT, int max_seq, cudaStream_t s);
 int smc_latent_attend(smc_ctx *, const smc_latent_dims &, const smc_latent_bufs &, const smc_rows &, int bf16, const smc_weight *w_ukv,
                       const float *sink, const float *cosT, const float *sinT, int max_seq, int pos0, cudaStream_t s);
-int smc_latent_reserve(smc_ctx *, const smc_latent_dims &, int max_batch);
+int smc_latent_check(smc_ctx *, const smc_latent_dims &);
 bool smc_latent_prefill_supported(const smc_latent_dims &);
+bool smc_latent_decode_supported(const smc_latent_dims &);  // the tensor-core form of the absorbed path (needs w_ukt)
+int smc_latent_transpose_uk(smc_ctx *, const smc_latent_dims &, const smc_weight *w_ukv, void *out, cudaStream_t s);
 // ---- state-space layers (smc_ssm.cu) ----
 struct smc_ssm_dims {
     int heads, vdim, state, groups, conv, norm_groups;
@@ -252,17 +259,13 @@ struct smc_ssm_bufs {
     int ld;
     const float *dt_raw;          // [rows, heads]
     void *xbc;                    // [rows, heads vdim + 2 groups state] after convolution and SiLU  T
-    float *dt;                    // [rows, heads]
     float *y;                     // [rows, heads vdim]
     void *o;                      // [rows, heads vdim]  T
     void *conv_state;             // [slots, conv, channels]  T: input of position p in row p % conv
     float *state;                 // [slots, heads, vdim, state]
-    float *work;                  // chunked pass: per chunk states and decays
-    size_t work_floats;
 };
 int smc_ssm_mix(smc_ctx *, const smc_ssm_dims &, const smc_ssm_bufs &, const smc_rows &, int bf16, const float *conv_w, const float *conv_b,
-                const float *dt_bias, const float *a_log, const float *d_skip, const float *norm, int pos0, cudaStream_t s);
-size_t smc_ssm_work_floats(const smc_ssm_dims &, int rows);
+                const float *dt_bias, const float *a_log, const float *d_skip, const float *norm, cudaStream_t s);
 // ---- layered models (smc_layered.cu) ----
 struct smc_layered;
 void smc_layered_free(smc_layered *);

@@ -47,16 +47,17 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1
 // contraction does not care which k a fragment register holds as long as both operands agree, so lane (g, q) takes the
 // 16 contiguous bytes k = 32 c + 8 q .. + 7 of weight rows g and g + 8 and of activation row g: every load is 16 bytes
 // wide and a row's four lanes read 64 contiguous bytes.  The first weight chunks are requested before the kernel waits
-// for its predecessor.
+// for its predecessor.  Grouped form (blockIdx.z = group): N rows per group, each group with its own columns of x.
 template <int NT, int U>
 __global__ void __launch_bounds__(256) dense_skinny_kernel(const bf16 *__restrict__ w, const bf16 *__restrict__ x, int ldx, int M, int N, int K,
-                                                           smc_dense_out o)
+                                                           smc_dense_out o, int x_group)
 {
     constexpr int TOK = NT * 8;
     __shared__ float red[8][16][TOK + 1];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, q = lane & 3;
-    const int n0 = blockIdx.x * 16, m0 = blockIdx.y * TOK;
+    const int n0 = blockIdx.x * 16, m0 = blockIdx.y * TOK, grp0 = blockIdx.z * N;
     const int chunks = (K + 31) >> 5;
+    w += (size_t)grp0 * K, x += (size_t)blockIdx.z * x_group;
     const bf16 *w0 = w + (size_t)min(n0 + g, N - 1) * K + 8 * q, *w1 = w + (size_t)min(n0 + g + 8, N - 1) * K + 8 * q;
     const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
     uint4 a0[U], a1[U];
@@ -118,7 +119,7 @@ __global__ void __launch_bounds__(256) dense_skinny_kernel(const bf16 *__restric
     } else {
         for (int e = threadIdx.x; e < 16 * TOK; e += 256) {
             const int r = e & 15, t = e >> 4;
-            if (m0 + t < M && n0 + r < N) put(o, m0 + t, n0 + r, total(r, t));
+            if (m0 + t < M && n0 + r < N) put(o, m0 + t, grp0 + n0 + r, total(r, t));
         }
     }
 }
@@ -440,9 +441,9 @@ int smc_launch_dense_rows(smc_ctx *ctx, const void *x, int x_bf16, int ldx, cons
         }
         const int nt = M <= 8 ? 1 : (M <= 16 ? 2 : 4);
         const dim3 grid((N + 15) / 16, (M + nt * 8 - 1) / (nt * 8));
-        if (nt == 1) smc_launch_dep(ctx->use_pdl, dense_skinny_kernel<1, 4>, grid, dim3(256), 0, s, w, xb, ldx, M, N, K, o);
-        else if (nt == 2) smc_launch_dep(ctx->use_pdl, dense_skinny_kernel<2, 4>, grid, dim3(256), 0, s, w, xb, ldx, M, N, K, o);
-        else smc_launch_dep(ctx->use_pdl, dense_skinny_kernel<4, 2>, grid, dim3(256), 0, s, w, xb, ldx, M, N, K, o);
+        if (nt == 1) smc_launch_dep(ctx->use_pdl, dense_skinny_kernel<1, 4>, grid, dim3(256), 0, s, w, xb, ldx, M, N, K, o, 0);
+        else if (nt == 2) smc_launch_dep(ctx->use_pdl, dense_skinny_kernel<2, 4>, grid, dim3(256), 0, s, w, xb, ldx, M, N, K, o, 0);
+        else smc_launch_dep(ctx->use_pdl, dense_skinny_kernel<4, 2>, grid, dim3(256), 0, s, w, xb, ldx, M, N, K, o, 0);
         SMC_LAUNCH_CHECK(ctx);
         return SMC_OK;
     }
@@ -457,6 +458,21 @@ int smc_launch_dense_rows(smc_ctx *ctx, const void *x, int x_bf16, int ldx, cons
     };
     if (x_bf16) go(static_cast<const bf16 *>(x));
     else go(static_cast<const float *>(x));
+    SMC_LAUNCH_CHECK(ctx);
+    return SMC_OK;
+}
+
+int smc_launch_dense_grouped(smc_ctx *ctx, const void *x, int ldx, int x_group, const void *w, int groups, int N, int K, int M, const smc_dense_out &o,
+                             cudaStream_t s)
+{
+    if (K % 8 || ldx % 8 || x_group % 8 || (reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(w) & 15))
+        return smc_fail(ctx, SMC_E_UNSUPPORTED, "grouped dense matmul: rows must start on 16-byte boundaries");
+    const bf16 *xb = static_cast<const bf16 *>(x), *wb = static_cast<const bf16 *>(w);
+    const int nt = M <= 8 ? 1 : (M <= 16 ? 2 : 4);
+    const dim3 grid((N + 15) / 16, (M + nt * 8 - 1) / (nt * 8), groups);
+    if (nt == 1) smc_launch_dep(ctx->use_pdl, dense_skinny_kernel<1, 4>, grid, dim3(256), 0, s, wb, xb, ldx, M, N, K, o, x_group);
+    else if (nt == 2) smc_launch_dep(ctx->use_pdl, dense_skinny_kernel<2, 4>, grid, dim3(256), 0, s, wb, xb, ldx, M, N, K, o, x_group);
+    else smc_launch_dep(ctx->use_pdl, dense_skinny_kernel<4, 2>, grid, dim3(256), 0, s, wb, xb, ldx, M, N, K, o, x_group);
     SMC_LAUNCH_CHECK(ctx);
     return SMC_OK;
 }

@@ -13,6 +13,7 @@
 #include <cuda_bf16.h>
 #include <math.h>
 
+#include <type_traits>
 #include <vector>
 
 #include "smc_common.cuh"
@@ -247,6 +248,209 @@ __device__ __forceinline__ uint32_t pack2(float a, float b)
     return *reinterpret_cast<const uint32_t *>(&v);
 }
 
+// ------------------------------------------------------------------------------ absorbed form on the tensor cores (bfloat16)
+// One row, up to 16 heads per cluster of eight CTAs; each CTA takes every eighth 64-key tile of the window and the cluster
+// merges its partial sums through distributed shared memory.  The absorbed query (fp32) enters as a bfloat16 pair hi + lo,
+// so scores keep 16 bits of it; the cached rows are exact operands of both products.  All heads read the same keys: a tile
+// is fetched once per 16 heads.
+//   shared memory: query planes [2][16][ldk], two key tiles [64][ldk], scores [16][66] fp32, weights [16][72] bfloat16
+constexpr int DT = 64, DCL = 8;
+template <int OPW>  // 16-column groups of the latent a warp accumulates (8 warps)
+__global__ void __cluster_dims__(DCL, 1, 1) __launch_bounds__(256)
+latent_decode_kernel(const float *__restrict__ qa, const bf16 *__restrict__ q, const bf16 *__restrict__ cache, bf16 *__restrict__ oc, smc_rows rw,
+                     const float *__restrict__ sink, const float *__restrict__ cosT, const float *__restrict__ sinT, int heads, int dim, int rk, int rd,
+                     int ring, int window, float scale, int max_seq)
+{
+    extern __shared__ __align__(16) uint8_t sm_raw[];
+    __shared__ float row_m[16], row_l[16], row_f[16], all_m[DCL][16], all_l[DCL][16], all_f[DCL][16];
+    const int row = rk + rd, row16 = (row + 15) & ~15, ldk = (row16 + 8) * 2;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, tg = lane & 3;
+    const int rank = blockIdx.x, h0 = blockIdx.y * 16, nh = min(16, heads - h0), r = blockIdx.z;
+    uint8_t *q_s = sm_raw, *k_s = q_s + 2 * 16 * ldk, *s_s = k_s + 2 * DT * ldk, *p_s = s_s + 16 * 66 * 4;
+    const uint32_t qb = (uint32_t)__cvta_generic_to_shared(q_s), kb = (uint32_t)__cvta_generic_to_shared(k_s), pb = (uint32_t)__cvta_generic_to_shared(p_s);
+    float *sc = reinterpret_cast<float *>(s_s);
+    for (uint32_t e = threadIdx.x; e < (uint32_t)((2 * 16 + 2 * DT) * ldk) / 16; e += 256) reinterpret_cast<uint4 *>(sm_raw)[e] = make_uint4(0u, 0u, 0u, 0u);
+    smc_grid_dep_sync();
+    __syncthreads();
+    int slot, p;
+    row_place(rw, r, slot, p);
+    const int lo = window > 0 ? max(0, p - window + 1) : 0, n = p - lo + 1, tiles = (n + DT - 1) / DT;
+    const bf16 *base = cache + (size_t)slot * ring * row;
+    const int chunks = row / 8;
+    auto fetch = [&](int t, int buf) {
+        for (int e = threadIdx.x; e < DT * chunks; e += 256) {
+            const int j = e / chunks, c = e % chunks, k = t * DT + j;
+            const bool in = k < n;
+            cp16(kb + (uint32_t)((buf * DT + j) * ldk + 16 * c), base + (size_t)((lo + (in ? k : 0)) % ring) * row + 8 * c, in);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    if (rank < tiles) fetch(rank, 0);
+    auto put_q = [&](int hh, int i, float v) {
+        const bf16 hi = __float2bfloat16_rn(v);
+        reinterpret_cast<bf16 *>(q_s + hh * ldk)[i] = hi;
+        reinterpret_cast<bf16 *>(q_s + (16 + hh) * ldk)[i] = __float2bfloat16_rn(v - __bfloat162float(hi));
+    };
+    for (int e = threadIdx.x; e < nh * rk; e += 256) put_q(e / rk, e % rk, qa[((size_t)r * heads + h0) * rk + e]);
+    const int half = rd / 2;
+    for (int e = threadIdx.x; e < nh * half; e += 256) {
+        const int hh = e / half, i = e % half;
+        const bf16 *src = q + ((size_t)r * heads + h0 + hh) * (dim + rd) + dim;
+        const size_t ti = (size_t)min(p, max_seq - 1) * half + i;
+        const float u = to_f(src[i]), v = to_f(src[half + i]), c = cosT[ti], s = sinT[ti];
+        put_q(hh, rk + i, __fsub_rn(__fmul_rn(u, c), __fmul_rn(v, s)));
+        put_q(hh, rk + half + i, __fadd_rn(__fmul_rn(v, c), __fmul_rn(u, s)));
+    }
+    if (threadIdx.x < 16) row_m[threadIdx.x] = -INFINITY, row_l[threadIdx.x] = 0.f;
+    float o[2 * OPW][4];
+#pragma unroll
+    for (int i = 0; i < 2 * OPW; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+    const uint32_t a_off = (uint32_t)(((lane & 7) + 8 * ((lane >> 3) & 1)) * ldk + 16 * (lane >> 4));
+    int buf = 0;
+    for (int t = rank; t < tiles; t += DCL, buf ^= 1) {
+        if (t + DCL < tiles) {
+            fetch(t + DCL, buf ^ 1);
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+        }
+        __syncthreads();
+        // ---- scores: eight keys per warp
+        {
+            float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+            // one ldmatrix brings the warp's eight keys for two k-steps
+            const uint32_t bk = kb + (uint32_t)((buf * DT + warp * 8 + (lane & 7)) * ldk + 16 * (lane >> 3));
+            for (int ks = 0; ks < row16 / 16; ks += 2) {
+                uint32_t b[4], ah[4], al[4];
+                ldsm4(bk + 32 * ks, b);  // (an odd last k-step reads the zero padding column group or the next row; unused)
+                ldsm4(qb + a_off + 32 * ks, ah);
+                ldsm4(qb + 16 * ldk + a_off + 32 * ks, al);
+                mma_bf16(s[0], ah, b[0], b[1]);
+                mma_bf16(s[1], al, b[0], b[1]);
+                if (ks + 1 < row16 / 16) {
+                    ldsm4(qb + a_off + 32 * ks + 32, ah);
+                    ldsm4(qb + 16 * ldk + a_off + 32 * ks + 32, al);
+                    mma_bf16(s[0], ah, b[2], b[3]);
+                    mma_bf16(s[1], al, b[2], b[3]);
+                }
+            }
+            const int key = warp * 8 + 2 * tg;
+            const bool i0 = t * DT + key < n, i1 = t * DT + key + 1 < n;
+            sc[g * 66 + key] = i0 ? (s[0][0] + s[1][0]) * scale : -INFINITY, sc[g * 66 + key + 1] = i1 ? (s[0][1] + s[1][1]) * scale : -INFINITY;
+            sc[(g + 8) * 66 + key] = i0 ? (s[0][2] + s[1][2]) * scale : -INFINITY, sc[(g + 8) * 66 + key + 1] = i1 ? (s[0][3] + s[1][3]) * scale : -INFINITY;
+        }
+        __syncthreads();
+        // ---- running softmax: two heads per warp
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const int hh = warp * 2 + i;
+            const float s0 = sc[hh * 66 + lane], s1 = sc[hh * 66 + lane + 32];
+            float m = fmaxf(s0, s1);
+#pragma unroll
+            for (int d = 16; d > 0; d >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, d));
+            m = fmaxf(m, row_m[hh]);  // every tile holds a key, so the maximum is finite
+            const float e0 = expf(s0 - m), e1 = expf(s1 - m);
+            const float l = smc_group_sum<32>(e0 + e1);
+            bf16 *pp = reinterpret_cast<bf16 *>(p_s) + hh * 72;
+            pp[lane] = __float2bfloat16_rn(e0), pp[lane + 32] = __float2bfloat16_rn(e1);
+            if (lane == 0) {
+                const float f = expf(row_m[hh] - m);
+                row_f[hh] = f, row_m[hh] = m, row_l[hh] = fmaf(row_l[hh], f, l);
+            }
+        }
+        __syncthreads();
+        const float f0 = row_f[g], f1 = row_f[g + 8];
+#pragma unroll
+        for (int i = 0; i < 2 * OPW; ++i) o[i][0] *= f0, o[i][1] *= f0, o[i][2] *= f1, o[i][3] *= f1;
+#pragma unroll
+        for (int ks = 0; ks < DT / 16; ++ks) {
+            uint32_t a[4];
+            ldsm4(pb + (uint32_t)(((lane & 7) + 8 * ((lane >> 3) & 1)) * 144 + 16 * (lane >> 4) + 32 * ks), a);
+#pragma unroll
+            for (int i = 0; i < OPW; ++i) {
+                const int grp = warp + 8 * i;
+                if (16 * grp < rk) {
+                    uint32_t b[4];
+                    ldsm4t(kb + (uint32_t)((buf * DT + ks * 16 + (lane & 7) + 8 * ((lane >> 3) & 1)) * ldk + 32 * grp + 16 * (lane >> 4)), b);
+                    mma_bf16(o[2 * i], a, b[0], b[1]);
+                    mma_bf16(o[2 * i + 1], a, b[2], b[3]);
+                }
+            }
+        }
+        __syncthreads();  // the tile buffer, scores and weights are rewritten next
+    }
+    // ---- merge over the cluster: partial sums [16][rk] fp32 over the key tiles' space
+    float *part = reinterpret_cast<float *>(k_s);
+    const int ldp = rk + 4;
+#pragma unroll
+    for (int i = 0; i < OPW; ++i) {
+        const int grp = warp + 8 * i;
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+            const int c = 16 * grp + 8 * j + 2 * tg;
+            if (c < rk) {
+                part[g * ldp + c] = o[2 * i + j][0], part[(g + 8) * ldp + c] = o[2 * i + j][2];
+                if (c + 1 < rk) part[g * ldp + c + 1] = o[2 * i + j][1], part[(g + 8) * ldp + c + 1] = o[2 * i + j][3];
+            }
+        }
+    }
+    auto cluster_sync = [] { asm volatile("barrier.cluster.arrive;\n\tbarrier.cluster.wait;" ::: "memory"); };
+    cluster_sync();
+    auto remote = [](const void *ptr, int cta) {
+        uint32_t a = (uint32_t)__cvta_generic_to_shared(ptr), v;
+        float f;
+        asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(v) : "r"(a), "r"(cta));
+        asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(f) : "r"(v) : "memory");
+        return f;
+    };
+    if (threadIdx.x < DCL * 16) {
+        const int k = threadIdx.x >> 4, hh = threadIdx.x & 15;
+        all_m[k][hh] = remote(&row_m[hh], k), all_l[k][hh] = remote(&row_l[hh], k);
+    }
+    __syncthreads();
+    if (threadIdx.x < 16) {
+        const int hh = threadIdx.x;
+        const float sk = sink && hh < nh ? sink[h0 + hh] : -INFINITY;
+        float top = sk;
+#pragma unroll
+        for (int k = 0; k < DCL; ++k) top = fmaxf(top, all_m[k][hh]);
+        float den = sink ? expf(sk - top) : 0.f;
+#pragma unroll
+        for (int k = 0; k < DCL; ++k) all_f[k][hh] = expf(all_m[k][hh] - top), den = fmaf(all_f[k][hh], all_l[k][hh], den);
+#pragma unroll
+        for (int k = 0; k < DCL; ++k) all_f[k][hh] = __fdiv_rn(all_f[k][hh], den);
+    }
+    __syncthreads();
+    const int per = (rk + DCL - 1) / DCL, c0 = rank * per, c1 = min(rk, c0 + per);
+    for (int e = threadIdx.x; e < nh * per; e += 256) {
+        const int hh = e / per, c = c0 + e % per;
+        if (c >= c1) continue;
+        float x[DCL], v = 0.f;
+#pragma unroll
+        for (int k = 0; k < DCL; ++k) x[k] = remote(&part[hh * ldp + c], k);  // zeros from a CTA without a tile, its factor is zero too
+#pragma unroll
+        for (int k = 0; k < DCL; ++k) v = fmaf(all_f[k][hh], x[k], v);
+        oc[((size_t)r * heads + h0 + hh) * rk + c] = __float2bfloat16_rn(v);
+    }
+    cluster_sync();  // nobody leaves while its sums are read
+}
+
+size_t decode_smem(const smc_latent_dims &d)
+{
+    const int row16 = (d.kv_rank + d.rot_dim + 15) & ~15, ldk = (row16 + 8) * 2;
+    const size_t tiles = (size_t)(2 * 16 + 2 * DT) * ldk, merged = (size_t)2 * 16 * ldk + (size_t)16 * (d.kv_rank + 4) * 4;
+    return (tiles > merged ? tiles : merged) + 16 * 66 * 4 + 16 * 72 * 2 + 64;
+}
+
+// ukt[h][c][d] = W_uk[h * dim + d][c]
+__global__ void __launch_bounds__(256) transpose_uk_kernel(const bf16 *__restrict__ wuk, bf16 *__restrict__ ukt, int heads, int dim, int rk)
+{
+    const size_t e = (size_t)blockIdx.x * 256 + threadIdx.x;
+    if (e >= (size_t)heads * dim * rk) return;
+    const int d = (int)(e % dim), c = (int)(e / dim % rk), h = (int)(e / ((size_t)dim * rk));
+    ukt[e] = wuk[((size_t)h * dim + d) * rk + c];
+}
+
 // 64 query rows of one head per CTA (16 per warp), key tiles of 64, two tile buffers filled by cp.async.  Scores and the
 // running softmax are fp32; the weights enter the second product as bfloat16.  Head sizes are padded to 16 with zeros in
 // shared memory.  VT: value tiles of 8 columns a thread keeps accumulators for.
@@ -408,21 +612,16 @@ size_t prefill_smem(const smc_latent_dims &d)
 constexpr int EXPAND_ROWS = 17;
 
 template <typename T>
-int attend_absorbed(smc_ctx *ctx, const smc_latent_dims &d, const smc_latent_bufs &b, const smc_rows &rw, const smc_weight *w_ukv, const float *sink,
-                    const float *cosT, const float *sinT, int max_seq, cudaStream_t s)
+int attend_rows(smc_ctx *ctx, const smc_latent_dims &d, const smc_latent_bufs &b, const smc_rows &rw, const float *sink, cudaStream_t s)
 {
-    const bf16 *wuk = reinterpret_cast<const bf16 *>(w_ukv->d_raw), *wuv = wuk + (size_t)d.heads * d.dim * d.kv_rank;
-    const int row = d.kv_rank + d.rot_dim, ny = (rw.n + 7) / 8;
-    smc_launch_dep(ctx->use_pdl, latent_absorb_kernel<T>, dim3(d.heads, (d.kv_rank + 63) / 64, ny), dim3(256), (size_t)8 * d.dim * sizeof(float), s,
-                   static_cast<const T *>(b.q), wuk, b.qa, rw, cosT, sinT, d.heads, d.dim, d.rot_dim, d.kv_rank, max_seq);
-    SMC_LAUNCH_CHECK(ctx);
+    const int row = d.kv_rank + d.rot_dim;
     const size_t smem = ((size_t)row + 8 * d.kv_rank) * sizeof(float);
 #define SMC_ATTEND(E)                                                                                                                        \
     do {                                                                                                                                     \
         if (smem > 40 * 1024)                                                                                                                \
             SMC_CUDA(ctx, cudaFuncSetAttribute(latent_attend_kernel<T, E>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));         \
         smc_launch_dep(ctx->use_pdl, latent_attend_kernel<T, E>, dim3(d.heads, rw.n), dim3(256), smem, s, (const float *)b.qa,               \
-                       static_cast<const T *>(b.cache), b.oc, rw, sink, d.heads, d.kv_rank, d.rot_dim, d.ring, d.window, d.scale);           \
+                       static_cast<const T *>(b.cache), static_cast<float *>(b.oc), rw, sink, d.heads, d.kv_rank, d.rot_dim, d.ring, d.window, d.scale);           \
     } while (0)
     if (d.kv_rank <= 64) SMC_ATTEND(2);
     else if (d.kv_rank <= 128) SMC_ATTEND(4);
@@ -431,7 +630,44 @@ int attend_absorbed(smc_ctx *ctx, const smc_latent_dims &d, const smc_latent_buf
     else SMC_ATTEND(32);
 #undef SMC_ATTEND
     SMC_LAUNCH_CHECK(ctx);
-    smc_launch_dep(ctx->use_pdl, latent_value_kernel<T>, dim3((d.heads * d.vdim + 7) / 8, ny), dim3(256), 0, s, (const float *)b.oc, wuv,
+    return SMC_OK;
+}
+
+// the same on the tensor cores: absorb, attend, rebuild the values
+int attend_absorbed_mma(smc_ctx *ctx, const smc_latent_dims &d, const smc_latent_bufs &b, const smc_rows &rw, const smc_weight *w_ukv, const float *sink,
+                        const float *cosT, const float *sinT, int max_seq, cudaStream_t s)
+{
+    smc_dense_out o{};
+    o.y = b.qa, o.ldy = d.heads * d.kv_rank;
+    int rc = smc_launch_dense_grouped(ctx, b.q, d.heads * (d.dim + d.rot_dim), d.dim + d.rot_dim, b.w_ukt, d.heads, d.kv_rank, d.dim, rw.n, o, s);
+    if (rc) return rc;
+    const size_t smem = decode_smem(d);
+    auto go = [&](auto kernel) {
+        SMC_CUDA(ctx, cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        smc_launch_dep(ctx->use_pdl, kernel, dim3(DCL, (d.heads + 15) / 16, rw.n), dim3(256), smem, s, (const float *)b.qa, (const bf16 *)b.q,
+                       (const bf16 *)b.cache, (bf16 *)b.oc, rw, sink, cosT, sinT, d.heads, d.dim, d.kv_rank, d.rot_dim, d.ring, d.window, d.scale, max_seq);
+        SMC_LAUNCH_CHECK(ctx);
+        return (int)SMC_OK;
+    };
+    rc = d.kv_rank <= 128 ? go(latent_decode_kernel<1>) : (d.kv_rank <= 256 ? go(latent_decode_kernel<2>) : go(latent_decode_kernel<4>));
+    if (rc) return rc;
+    o.y = b.o, o.ldy = d.heads * d.vdim, o.y_bf16 = 1;
+    const bf16 *wuv = reinterpret_cast<const bf16 *>(w_ukv->d_raw) + (size_t)d.heads * d.dim * d.kv_rank;
+    return smc_launch_dense_grouped(ctx, b.oc, d.heads * d.kv_rank, d.kv_rank, wuv, d.heads, d.vdim, d.kv_rank, rw.n, o, s);
+}
+
+template <typename T>
+int attend_absorbed(smc_ctx *ctx, const smc_latent_dims &d, const smc_latent_bufs &b, const smc_rows &rw, const smc_weight *w_ukv, const float *sink,
+                    const float *cosT, const float *sinT, int max_seq, cudaStream_t s)
+{
+    const bf16 *wuk = reinterpret_cast<const bf16 *>(w_ukv->d_raw), *wuv = wuk + (size_t)d.heads * d.dim * d.kv_rank;
+    const int ny = (rw.n + 7) / 8;
+    smc_launch_dep(ctx->use_pdl, latent_absorb_kernel<T>, dim3(d.heads, (d.kv_rank + 63) / 64, ny), dim3(256), (size_t)8 * d.dim * sizeof(float), s,
+                   static_cast<const T *>(b.q), wuk, b.qa, rw, cosT, sinT, d.heads, d.dim, d.rot_dim, d.kv_rank, max_seq);
+    SMC_LAUNCH_CHECK(ctx);
+    int rc = attend_rows<T>(ctx, d, b, rw, sink, s);
+    if (rc) return rc;
+    smc_launch_dep(ctx->use_pdl, latent_value_kernel<T>, dim3((d.heads * d.vdim + 7) / 8, ny), dim3(256), 0, s, static_cast<const float *>(b.oc), wuv,
                    static_cast<T *>(b.o), rw.n, d.heads, d.vdim, d.kv_rank);
     SMC_LAUNCH_CHECK(ctx);
     return SMC_OK;
@@ -444,9 +680,22 @@ bool smc_latent_prefill_supported(const smc_latent_dims &d)
     return d.dim % 8 == 0 && d.rot_dim % 8 == 0 && d.vdim % 8 == 0 && d.kv_rank % 8 == 0 && d.vdim <= 256 && prefill_smem(d) <= 220 * 1024;
 }
 
-int smc_latent_reserve(smc_ctx *ctx, const smc_latent_dims &d, int max_batch)
+bool smc_latent_decode_supported(const smc_latent_dims &d)
 {
-    (void)max_batch;
+    return d.dim % 8 == 0 && d.kv_rank % 8 == 0 && d.rot_dim % 8 == 0 && d.kv_rank <= 512 && decode_smem(d) <= 220 * 1024;
+}
+
+int smc_latent_transpose_uk(smc_ctx *ctx, const smc_latent_dims &d, const smc_weight *w_ukv, void *out, cudaStream_t s)
+{
+    const size_t n = (size_t)d.heads * d.dim * d.kv_rank;
+    transpose_uk_kernel<<<(unsigned)((n + 255) / 256), 256, 0, s>>>(reinterpret_cast<const bf16 *>(w_ukv->d_raw), static_cast<bf16 *>(out), d.heads, d.dim,
+                                                                   d.kv_rank);
+    SMC_LAUNCH_CHECK(ctx);
+    return SMC_OK;
+}
+
+int smc_latent_check(smc_ctx *ctx, const smc_latent_dims &d)
+{
     if (d.kv_rank > 1024) return smc_fail(ctx, SMC_E_UNSUPPORTED, "latent attention: kv_rank %d (up to 1024 are built)", d.kv_rank);
     if (d.rot_dim % 2) return smc_fail(ctx, SMC_E_UNSUPPORTED, "latent attention: an odd rotated part of %d", d.rot_dim);
     if (d.dim > 1024) return smc_fail(ctx, SMC_E_UNSUPPORTED, "latent attention: dim %d (up to 1024 are built)", d.dim);
@@ -472,8 +721,10 @@ int smc_latent_attend(smc_ctx *ctx, const smc_latent_dims &d, const smc_latent_b
                       const float *sink, const float *cosT, const float *sinT, int max_seq, int pos0, cudaStream_t s)
 {
     if (!is_bf16) return attend_absorbed<float>(ctx, d, b, rw, w_ukv, sink, cosT, sinT, max_seq, s);
-    if (rw.seq0 < 0 || rw.n < EXPAND_ROWS || !smc_latent_prefill_supported(d))
+    if (rw.seq0 < 0 || rw.n < EXPAND_ROWS || !smc_latent_prefill_supported(d)) {
+        if (b.w_ukt && smc_latent_decode_supported(d)) return attend_absorbed_mma(ctx, d, b, rw, w_ukv, sink, cosT, sinT, max_seq, s);
         return attend_absorbed<bf16>(ctx, d, b, rw, w_ukv, sink, cosT, sinT, max_seq, s);
+    }
     // expanded: the visible rows in order, their keys and values per head, then the tensor cores
     const int k0 = d.window > 0 && pos0 > d.window - 1 ? pos0 - d.window + 1 : 0, nk = pos0 + rw.n - k0, row = d.kv_rank + d.rot_dim;
     const int row16 = row / 8;

@@ -6,6 +6,7 @@
 // convolution inputs.  Positions live on the device (a captured step can advance them itself, SMC_POS_NEXT); the host
 // keeps its own count where it knows it and refuses a call that would continue a recurrence at another place.
 #include <algorithm>
+#include <utility>
 #include <vector>
 
 #include "smc_common.cuh"
@@ -23,6 +24,7 @@ struct smc_layered {
         float *ssm = nullptr;
         int ring_rows = 0;
         const float *cosT = nullptr, *sinT = nullptr;
+        const void *ukt = nullptr;
     };
     std::vector<State> state;
     struct Table {
@@ -30,8 +32,9 @@ struct smc_layered {
         float *c, *s;
     };
     std::vector<Table> tables;  // layers with the same rotation share one
-    float *x = nullptr, *y = nullptr, *qa = nullptr, *oc = nullptr, *dt_raw = nullptr, *ssm_y = nullptr, *work = nullptr;
-    size_t work_floats = 0;
+    std::vector<std::pair<const smc_weight *, void *>> ukt;  // transposed key expansions, one per weight
+    void *oc = nullptr;
+    float *x = nullptr, *y = nullptr, *qa = nullptr, *dt_raw = nullptr, *ssm_y = nullptr;
     void *x16 = nullptr, *wide = nullptr, *cq = nullptr, *q = nullptr, *o = nullptr, *keys = nullptr, *kv = nullptr, *xbc = nullptr, *act = nullptr,
          *head = nullptr;
     float *dump = nullptr;
@@ -64,7 +67,7 @@ int check_layer(smc_ctx *ctx, const smc_layered_desc &d, const smc_layer_desc &L
             !shape_is(L.w_ukv, (long long)L.heads * (L.dim + L.vdim), L.kv_rank))
             return bad("latent attention weight shapes");
         smc_latent_dims ld{L.heads, L.dim, L.rot_dim, L.vdim, L.q_rank, L.kv_rank, L.window, 0, L.scale, d.eps};
-        int rc = smc_latent_reserve(ctx, ld, 1);
+        int rc = smc_latent_check(ctx, ld);
         if (rc) return rc;
     } else if (L.mixer == SMC_MIX_MAMBA2) {
         if (L.state <= 0 || L.groups <= 0 || L.heads % L.groups || L.conv <= 0 || L.norm_groups <= 0 || (L.heads * L.vdim) % L.norm_groups || !L.conv_w ||
@@ -91,7 +94,8 @@ void smc_layered_free(smc_layered *m)
     if (!m) return;
     for (auto &s : m->state) cudaFree(s.ring), cudaFree(s.conv), cudaFree(s.ssm);
     for (auto &t : m->tables) cudaFree(t.c), cudaFree(t.s);
-    void *bufs[] = {m->pos, m->x, m->y, m->qa, m->oc, m->dt_raw, m->ssm_y, m->work, m->x16, m->wide, m->cq, m->q, m->o, m->keys, m->kv, m->xbc, m->act, m->head};
+    for (auto &t : m->ukt) cudaFree(t.second);
+    void *bufs[] = {m->pos, m->x, m->y, m->qa, m->oc, m->dt_raw, m->ssm_y, m->x16, m->wide, m->cq, m->q, m->o, m->keys, m->kv, m->xbc, m->act, m->head};
     for (void *p : bufs) cudaFree(p);
     delete m;
 }
@@ -153,12 +157,22 @@ int smc_layered_create(smc_ctx *ctx, const smc_layered_desc *desc, int max_batch
                 it = m->tables.end() - 1;
             }
             st.cosT = it->c, st.sinT = it->s;
+            if (m->bf16 && smc_latent_decode_supported(latent_dims(m, l))) {
+                auto u = std::find_if(m->ukt.begin(), m->ukt.end(), [&](auto &t) { return t.first == L.w_ukv; });
+                if (u == m->ukt.end()) {
+                    void *t = nullptr;
+                    alloc(&t, (size_t)L.heads * L.dim * L.kv_rank * 2);
+                    m->ukt.emplace_back(L.w_ukv, t);
+                    if (e == cudaSuccess && !rc) rc = smc_latent_transpose_uk(ctx, latent_dims(m, l), L.w_ukv, t, ctx->stream);
+                    u = m->ukt.end() - 1;
+                }
+                st.ukt = u->second;
+            }
         } else {
             const size_t inner = (size_t)L.heads * L.vdim, ch = inner + 2 * (size_t)L.groups * L.state;
             alloc(&st.conv, B * L.conv * ch * el, true);
             alloc(&st.ssm, B * inner * L.state * sizeof(float), true);
             wide = std::max(wide, inner + ch), dt = std::max(dt, (size_t)L.heads), xbc = std::max(xbc, ch), sy = std::max(sy, inner);
-            m->work_floats = std::max(m->work_floats, smc_ssm_work_floats(ssm_dims(m, L), m->rows));
         }
         if (rc || e != cudaSuccess) break;
     }
@@ -166,12 +180,13 @@ int smc_layered_create(smc_ctx *ctx, const smc_layered_desc *desc, int max_batch
     alloc(&m->x, R * d.hidden * 4), alloc(&m->y, R * d.hidden * 4), alloc(&m->x16, m->bf16 ? R * d.hidden * 2 : 0), alloc(&m->head, R * d.hidden * el);
     alloc(&m->wide, R * wide * el), alloc(&m->cq, R * cq * el), alloc(&m->q, R * q * el), alloc(&m->qa, R * qa * 4), alloc(&m->oc, R * oc * 4);
     alloc(&m->o, R * o * el), alloc(&m->keys, keys * el), alloc(&m->kv, kv * el), alloc(&m->dt_raw, R * dt * 4), alloc(&m->xbc, R * xbc * el);
-    alloc(&m->ssm_y, R * sy * 4), alloc(&m->act, R * act * el), alloc(&m->work, m->work_floats * 4);
+    alloc(&m->ssm_y, R * sy * 4), alloc(&m->act, R * act * el);
     if (e != cudaSuccess && !rc) rc = smc_fail(ctx, SMC_E_CUDA, "model_create_layered: allocation failed: %s", cudaGetErrorString(e));
     if (rc) {
         smc_layered_free(m);
         return rc;
     }
+    SMC_CUDA(ctx, cudaStreamSynchronize(ctx->stream));
     *out = m;
     return SMC_OK;
 }
@@ -213,7 +228,7 @@ int smc_layered_forward(smc_ctx *ctx, smc_layered *m, const int *d_tokens, int c
         smc_layered::State &st = m->state[l];
         if (L.mixer == SMC_MIX_LATENT) {
             const smc_latent_dims ld = latent_dims(m, l);
-            const smc_latent_bufs lb{m->wide, m->cq, m->q, m->qa, m->oc, m->o, m->keys, m->kv, st.ring};
+            const smc_latent_bufs lb{m->wide, m->cq, m->q, m->qa, m->oc, st.ukt, m->o, m->keys, m->kv, st.ring};
             SMC_TRY(smc_launch_dense(ctx, xin, bf, H, L.w_down, n, to(m->wide, L.w_down->N, bf), s));
             SMC_TRY(smc_latent_post(ctx, ld, lb, rw, bf, L.q_norm, L.kv_norm, st.cosT, st.sinT, d.max_seq, s));
             SMC_TRY(smc_launch_dense(ctx, m->cq, bf, L.q_rank, L.w_uq, n, to(m->q, L.w_uq->N, bf), s));
@@ -223,8 +238,8 @@ int smc_layered_forward(smc_ctx *ctx, smc_layered *m, const int *d_tokens, int c
             smc_dense_out out = to(m->wide, ld, bf);
             out.y32 = m->dt_raw, out.ld32 = L.heads, out.split = ld;  // step sizes stay fp32
             SMC_TRY(smc_launch_dense(ctx, xin, bf, H, L.w_in, n, out, s));
-            const smc_ssm_bufs sb{m->wide, ld, m->dt_raw, m->xbc, nullptr, m->ssm_y, m->o, st.conv, st.ssm, m->work, m->work_floats};
-            SMC_TRY(smc_ssm_mix(ctx, ssm_dims(m, L), sb, rw, bf, L.conv_w, L.conv_b, L.dt_bias, L.a_log, L.d_skip, L.mix_norm, pos, s));
+            const smc_ssm_bufs sb{m->wide, ld, m->dt_raw, m->xbc, m->ssm_y, m->o, st.conv, st.ssm};
+            SMC_TRY(smc_ssm_mix(ctx, ssm_dims(m, L), sb, rw, bf, L.conv_w, L.conv_b, L.dt_bias, L.a_log, L.d_skip, L.mix_norm, s));
         }
         SMC_TRY(smc_launch_dense(ctx, m->o, bf, L.heads * L.vdim, L.w_out, n, to(m->y, H, 0), s));
         SMC_TRY(smc_scaled_add_rmsnorm_dev(ctx, m->x, m->y, L.norm1, m->x16, n, H, d.alpha, 1.0f, d.eps, s));
