@@ -48,14 +48,15 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1
 // 16 contiguous bytes k = 32 c + 8 q .. + 7 of weight rows g and g + 8 and of activation row g: every load is 16 bytes
 // wide and a row's four lanes read 64 contiguous bytes.  The first weight chunks are requested before the kernel waits
 // for its predecessor.  Grouped form (blockIdx.z = group): N rows per group, each group with its own columns of x.
-template <int NT, int U>
+// HALF: eight weight rows per CTA (the upper half of each fragment is zero), for matrices with too few rows to fill the SMs.
+template <int NT, int U, bool HALF>
 __global__ void __launch_bounds__(256) dense_skinny_kernel(const bf16 *__restrict__ w, const bf16 *__restrict__ x, int ldx, int M, int N, int K,
                                                            smc_dense_out o, int x_group)
 {
-    constexpr int TOK = NT * 8;
-    __shared__ float red[8][16][TOK + 1];
+    constexpr int TOK = NT * 8, ROWS = HALF ? 8 : 16;
+    __shared__ float red[8][ROWS][TOK + 1];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, q = lane & 3;
-    const int n0 = blockIdx.x * 16, m0 = blockIdx.y * TOK, grp0 = blockIdx.z * N;
+    const int n0 = blockIdx.x * ROWS, m0 = blockIdx.y * TOK, grp0 = blockIdx.z * N;
     const int chunks = (K + 31) >> 5;
     w += (size_t)grp0 * K, x += (size_t)blockIdx.z * x_group;
     const bf16 *w0 = w + (size_t)min(n0 + g, N - 1) * K + 8 * q, *w1 = w + (size_t)min(n0 + g + 8, N - 1) * K + 8 * q;
@@ -67,7 +68,7 @@ __global__ void __launch_bounds__(256) dense_skinny_kernel(const bf16 *__restric
             const int c = c0 + 8 * u;
             const bool in = c < chunks && 32 * c + 8 * q < K;
             a0[u] = in ? smc_ldg_stream16(w0 + 32 * c) : zero;
-            a1[u] = in ? smc_ldg_stream16(w1 + 32 * c) : zero;
+            a1[u] = in && !HALF ? smc_ldg_stream16(w1 + 32 * c) : zero;
         }
     };
     fetch(warp);
@@ -102,7 +103,7 @@ __global__ void __launch_bounds__(256) dense_skinny_kernel(const bf16 *__restric
 #pragma unroll
     for (int t = 0; t < NT; ++t) {
         red[warp][g][8 * t + 2 * q] = acc[t][0], red[warp][g][8 * t + 2 * q + 1] = acc[t][1];
-        red[warp][g + 8][8 * t + 2 * q] = acc[t][2], red[warp][g + 8][8 * t + 2 * q + 1] = acc[t][3];
+        if (!HALF) red[warp][g + ROWS - 8][8 * t + 2 * q] = acc[t][2], red[warp][g + ROWS - 8][8 * t + 2 * q + 1] = acc[t][3];
     }
     __syncthreads();
     auto total = [&](int r, int t) {
@@ -112,13 +113,13 @@ __global__ void __launch_bounds__(256) dense_skinny_kernel(const bf16 *__restric
         return v;
     };
     if (o.woven) {
-        for (int e = threadIdx.x; e < 8 * TOK; e += 256) {
-            const int i = e & 7, t = e >> 3;
+        for (int e = threadIdx.x; e < ROWS / 2 * TOK; e += 256) {
+            const int i = e % (ROWS / 2), t = e / (ROWS / 2);
             if (m0 + t < M && n0 + 2 * i + 1 < N) put_pair(o, m0 + t, (n0 >> 1) + i, total(2 * i, t), total(2 * i + 1, t));
         }
     } else {
-        for (int e = threadIdx.x; e < 16 * TOK; e += 256) {
-            const int r = e & 15, t = e >> 4;
+        for (int e = threadIdx.x; e < ROWS * TOK; e += 256) {
+            const int r = e % ROWS, t = e / ROWS;
             if (m0 + t < M && n0 + r < N) put(o, m0 + t, grp0 + n0 + r, total(r, t));
         }
     }
@@ -407,6 +408,19 @@ int launch_tc(smc_ctx *ctx, const bf16 *x, int ldx, const bf16 *w, int M, int N,
     return SMC_OK;
 }
 
+void launch_skinny(smc_ctx *ctx, const bf16 *x, int ldx, int x_group, const bf16 *w, int groups, int N, int K, int M, const smc_dense_out &o, cudaStream_t s)
+{
+    const int nt = M <= 8 ? 1 : (M <= 16 ? 2 : 4), my = (M + nt * 8 - 1) / (nt * 8);
+    const bool half = (long long)((N + 15) / 16) * my * groups < 2 * ctx->sm_count;  // fewer than two CTAs per SM
+    const dim3 grid(half ? (N + 7) / 8 : (N + 15) / 16, my, groups);
+    auto go = [&](auto kernel) { smc_launch_dep(ctx->use_pdl, kernel, grid, dim3(256), 0, s, w, x, ldx, M, N, K, o, x_group); };
+    const bool deep = K >= 2048;  // eight chunks and more per warp
+    if (nt == 1 && deep) half ? go(dense_skinny_kernel<1, 8, true>) : go(dense_skinny_kernel<1, 8, false>);
+    else if (nt == 1) half ? go(dense_skinny_kernel<1, 4, true>) : go(dense_skinny_kernel<1, 4, false>);
+    else if (nt == 2) half ? go(dense_skinny_kernel<2, 4, true>) : go(dense_skinny_kernel<2, 4, false>);
+    else half ? go(dense_skinny_kernel<4, 4, true>) : go(dense_skinny_kernel<4, 4, false>);
+}
+
 __global__ void __launch_bounds__(256) round_bf16_kernel(const float *__restrict__ x, bf16 *__restrict__ y, long long n)
 {
     smc_grid_dep_sync();
@@ -439,11 +453,7 @@ int smc_launch_dense_rows(smc_ctx *ctx, const void *x, int x_bf16, int ldx, cons
             if ((long long)mt * ((N + 255) / 256) >= ctx->sm_count) return launch_tc<256>(ctx, xb, ldx, w, M, N, K, o, s);
             return launch_tc<128>(ctx, xb, ldx, w, M, N, K, o, s);
         }
-        const int nt = M <= 8 ? 1 : (M <= 16 ? 2 : 4);
-        const dim3 grid((N + 15) / 16, (M + nt * 8 - 1) / (nt * 8));
-        if (nt == 1) smc_launch_dep(ctx->use_pdl, dense_skinny_kernel<1, 4>, grid, dim3(256), 0, s, w, xb, ldx, M, N, K, o, 0);
-        else if (nt == 2) smc_launch_dep(ctx->use_pdl, dense_skinny_kernel<2, 4>, grid, dim3(256), 0, s, w, xb, ldx, M, N, K, o, 0);
-        else smc_launch_dep(ctx->use_pdl, dense_skinny_kernel<4, 2>, grid, dim3(256), 0, s, w, xb, ldx, M, N, K, o, 0);
+        launch_skinny(ctx, xb, ldx, 0, w, 1, N, K, M, o, s);
         SMC_LAUNCH_CHECK(ctx);
         return SMC_OK;
     }
@@ -468,11 +478,7 @@ int smc_launch_dense_grouped(smc_ctx *ctx, const void *x, int ldx, int x_group, 
     if (K % 8 || ldx % 8 || x_group % 8 || (reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(w) & 15))
         return smc_fail(ctx, SMC_E_UNSUPPORTED, "grouped dense matmul: rows must start on 16-byte boundaries");
     const bf16 *xb = static_cast<const bf16 *>(x), *wb = static_cast<const bf16 *>(w);
-    const int nt = M <= 8 ? 1 : (M <= 16 ? 2 : 4);
-    const dim3 grid((N + 15) / 16, (M + nt * 8 - 1) / (nt * 8), groups);
-    if (nt == 1) smc_launch_dep(ctx->use_pdl, dense_skinny_kernel<1, 4>, grid, dim3(256), 0, s, wb, xb, ldx, M, N, K, o, x_group);
-    else if (nt == 2) smc_launch_dep(ctx->use_pdl, dense_skinny_kernel<2, 4>, grid, dim3(256), 0, s, wb, xb, ldx, M, N, K, o, x_group);
-    else smc_launch_dep(ctx->use_pdl, dense_skinny_kernel<4, 2>, grid, dim3(256), 0, s, wb, xb, ldx, M, N, K, o, x_group);
+    launch_skinny(ctx, xb, ldx, x_group, wb, groups, N, K, M, o, s);
     SMC_LAUNCH_CHECK(ctx);
     return SMC_OK;
 }

@@ -517,26 +517,53 @@ int ew_grid(long long items, int cap)
 
 // x = alpha * x + y, then x = x / rms(x) * (w_offset + w): the norm AFTER the residual sum, in place on the fp32 stream,
 // with an optional bfloat16 copy for the matmuls that read it.  A CTA per row; the sum stays in shared memory.
+template <bool VEC>
 __global__ void __launch_bounds__(256) scaled_add_rmsnorm_kernel(float *x, const float *__restrict__ y, const float *__restrict__ w,
                                                                  __nv_bfloat16 *__restrict__ x16, int n, float alpha, float w_offset, float eps)
 {
-    extern __shared__ float row_s[];
+    extern __shared__ __align__(16) float row_s[];
     __shared__ float red[32];
     smc_grid_dep_sync();
     float *p = x + (size_t)blockIdx.x * n;
     const float *q = y ? y + (size_t)blockIdx.x * n : nullptr;
+    __nv_bfloat16 *o = x16 ? x16 + (size_t)blockIdx.x * n : nullptr;
     float ss = 0.f;
-    for (int i = threadIdx.x; i < n; i += blockDim.x) {
-        const float v = q ? fmaf(alpha, p[i], q[i]) : alpha * p[i];
-        row_s[i] = v;
-        ss = fmaf(v, v, ss);
+    if (VEC) {
+        const float4 *p4 = reinterpret_cast<const float4 *>(p), *q4 = reinterpret_cast<const float4 *>(q);
+#pragma unroll 2
+        for (int i = threadIdx.x; i < n / 4; i += blockDim.x) {
+            const float4 a = p4[i], b = q ? q4[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+            const float4 v = make_float4(fmaf(alpha, a.x, b.x), fmaf(alpha, a.y, b.y), fmaf(alpha, a.z, b.z), fmaf(alpha, a.w, b.w));
+            reinterpret_cast<float4 *>(row_s)[i] = v;
+            ss = fmaf(v.x, v.x, ss), ss = fmaf(v.y, v.y, ss), ss = fmaf(v.z, v.z, ss), ss = fmaf(v.w, v.w, ss);
+        }
+    } else {
+        for (int i = threadIdx.x; i < n; i += blockDim.x) {
+            const float v = q ? fmaf(alpha, p[i], q[i]) : alpha * p[i];
+            row_s[i] = v;
+            ss = fmaf(v, v, ss);
+        }
     }
     ss = block_sum(ss, red);
     const float inv = __fdiv_rn(1.0f, sqrtf(__fdiv_rn(ss, (float)n) + eps));
-    for (int i = threadIdx.x; i < n; i += blockDim.x) {
-        const float v = (row_s[i] * inv) * (w_offset + w[i]);
-        p[i] = v;
-        if (x16) x16[(size_t)blockIdx.x * n + i] = __float2bfloat16_rn(v);
+    if (VEC) {
+#pragma unroll 2
+        for (int i = threadIdx.x; i < n / 4; i += blockDim.x) {
+            const float4 v = reinterpret_cast<const float4 *>(row_s)[i], g = __ldg(reinterpret_cast<const float4 *>(w) + i);
+            const float4 r = make_float4((v.x * inv) * (w_offset + g.x), (v.y * inv) * (w_offset + g.y), (v.z * inv) * (w_offset + g.z),
+                                         (v.w * inv) * (w_offset + g.w));
+            reinterpret_cast<float4 *>(p)[i] = r;
+            if (o) {
+                const __nv_bfloat162 lo = __floats2bfloat162_rn(r.x, r.y), hi = __floats2bfloat162_rn(r.z, r.w);
+                reinterpret_cast<uint2 *>(o)[i] = make_uint2(*reinterpret_cast<const uint32_t *>(&lo), *reinterpret_cast<const uint32_t *>(&hi));
+            }
+        }
+    } else {
+        for (int i = threadIdx.x; i < n; i += blockDim.x) {
+            const float v = (row_s[i] * inv) * (w_offset + w[i]);
+            p[i] = v;
+            if (o) o[i] = __float2bfloat16_rn(v);
+        }
     }
 }
 
@@ -820,10 +847,15 @@ int smc_scaled_add_rmsnorm_dev(smc_ctx *ctx, float *d_x, const float *d_y, const
     const size_t smem = (size_t)n * sizeof(float);
     if (smem > 200 * 1024) return smc_fail(ctx, SMC_E_UNSUPPORTED, "scaled_add_rmsnorm: rows of %d elements", n);
     if (rows == 0) return SMC_OK;
-    if (smem > 40 * 1024)
-        SMC_CUDA(ctx, cudaFuncSetAttribute(scaled_add_rmsnorm_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    smc_launch_dep(ctx->use_pdl, scaled_add_rmsnorm_kernel, dim3(rows), dim3(256), smem, static_cast<cudaStream_t>(stream), d_x, d_y, d_w,
-                   static_cast<__nv_bfloat16 *>(d_x16), n, alpha, w_offset, eps);
+    const bool vec = n % 4 == 0 && ((reinterpret_cast<uintptr_t>(d_x) | reinterpret_cast<uintptr_t>(d_y) | reinterpret_cast<uintptr_t>(d_w) |
+                                     reinterpret_cast<uintptr_t>(d_x16)) & 15) == 0;
+    auto go = [&](auto kernel) {
+        if (smem > 40 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        smc_launch_dep(ctx->use_pdl, kernel, dim3(rows), dim3(256), smem, static_cast<cudaStream_t>(stream), d_x, d_y, d_w,
+                       static_cast<__nv_bfloat16 *>(d_x16), n, alpha, w_offset, eps);
+    };
+    if (vec) go(scaled_add_rmsnorm_kernel<true>);
+    else go(scaled_add_rmsnorm_kernel<false>);
     SMC_LAUNCH_CHECK(ctx);
     return SMC_OK;
 }

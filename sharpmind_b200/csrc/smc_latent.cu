@@ -249,14 +249,16 @@ __device__ __forceinline__ uint32_t pack2(float a, float b)
 }
 
 // ------------------------------------------------------------------------------ absorbed form on the tensor cores (bfloat16)
-// One row, up to 16 heads per cluster of eight CTAs; each CTA takes every eighth 64-key tile of the window and the cluster
-// merges its partial sums through distributed shared memory.  The absorbed query (fp32) enters as a bfloat16 pair hi + lo,
+// One row, up to 16 heads per cluster of up to eight CTAs; each CTA takes every cluster-size-th 64-key tile of the window and
+// the cluster merges its partial sums through distributed shared memory.  The absorbed query (fp32) enters as a bfloat16 pair hi + lo,
 // so scores keep 16 bits of it; the cached rows are exact operands of both products.  All heads read the same keys: a tile
 // is fetched once per 16 heads.
 //   shared memory: query planes [2][16][ldk], two key tiles [64][ldk], scores [16][66] fp32, weights [16][72] bfloat16
+// The keys and the position are fetched BEFORE the wait for the predecessor: they were written by the kernel before it, and a
+// kernel that is launched early is so only after every CTA of its predecessor has passed its own wait.
 constexpr int DT = 64, DCL = 8;
 template <int OPW>  // 16-column groups of the latent a warp accumulates (8 warps)
-__global__ void __cluster_dims__(DCL, 1, 1) __launch_bounds__(256)
+__global__ void __launch_bounds__(256)
 latent_decode_kernel(const float *__restrict__ qa, const bf16 *__restrict__ q, const bf16 *__restrict__ cache, bf16 *__restrict__ oc, smc_rows rw,
                      const float *__restrict__ sink, const float *__restrict__ cosT, const float *__restrict__ sinT, int heads, int dim, int rk, int rd,
                      int ring, int window, float scale, int max_seq)
@@ -269,9 +271,14 @@ latent_decode_kernel(const float *__restrict__ qa, const bf16 *__restrict__ q, c
     uint8_t *q_s = sm_raw, *k_s = q_s + 2 * 16 * ldk, *s_s = k_s + 2 * DT * ldk, *p_s = s_s + 16 * 66 * 4;
     const uint32_t qb = (uint32_t)__cvta_generic_to_shared(q_s), kb = (uint32_t)__cvta_generic_to_shared(k_s), pb = (uint32_t)__cvta_generic_to_shared(p_s);
     float *sc = reinterpret_cast<float *>(s_s);
-    for (uint32_t e = threadIdx.x; e < (uint32_t)((2 * 16 + 2 * DT) * ldk) / 16; e += 256) reinterpret_cast<uint4 *>(sm_raw)[e] = make_uint4(0u, 0u, 0u, 0u);
-    smc_grid_dep_sync();
-    __syncthreads();
+    const int cl = gridDim.x;
+    // padding columns of the planes and tiles, and the planes' rows without a head
+    const int pad = ldk / 2 - row;
+    for (int e = threadIdx.x; e < (2 * 16 + 2 * DT) * pad; e += 256) reinterpret_cast<bf16 *>(sm_raw + (e / pad) * ldk)[row + e % pad] = __float2bfloat16_rn(0.f);
+    for (int e = threadIdx.x; e < 2 * (16 - nh) * row; e += 256) {
+        const int rr = e / row, pl = rr / (16 - nh);
+        reinterpret_cast<bf16 *>(sm_raw + (pl * 16 + nh + rr % (16 - nh)) * ldk)[e % row] = __float2bfloat16_rn(0.f);
+    }
     int slot, p;
     row_place(rw, r, slot, p);
     const int lo = window > 0 ? max(0, p - window + 1) : 0, n = p - lo + 1, tiles = (n + DT - 1) / DT;
@@ -286,6 +293,7 @@ latent_decode_kernel(const float *__restrict__ qa, const bf16 *__restrict__ q, c
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     if (rank < tiles) fetch(rank, 0);
+    smc_grid_dep_sync();
     auto put_q = [&](int hh, int i, float v) {
         const bf16 hi = __float2bfloat16_rn(v);
         reinterpret_cast<bf16 *>(q_s + hh * ldk)[i] = hi;
@@ -307,9 +315,9 @@ latent_decode_kernel(const float *__restrict__ qa, const bf16 *__restrict__ q, c
     for (int i = 0; i < 2 * OPW; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     const uint32_t a_off = (uint32_t)(((lane & 7) + 8 * ((lane >> 3) & 1)) * ldk + 16 * (lane >> 4));
     int buf = 0;
-    for (int t = rank; t < tiles; t += DCL, buf ^= 1) {
-        if (t + DCL < tiles) {
-            fetch(t + DCL, buf ^ 1);
+    for (int t = rank; t < tiles; t += cl, buf ^= 1) {
+        if (t + cl < tiles) {
+            fetch(t + cl, buf ^ 1);
             asm volatile("cp.async.wait_group 1;" ::: "memory");
         } else {
             asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -317,12 +325,15 @@ latent_decode_kernel(const float *__restrict__ qa, const bf16 *__restrict__ q, c
         __syncthreads();
         // ---- scores: eight keys per warp
         {
-            float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+            float s[4][4];  // hi and lo of even and odd k-steps: four chains of dependent products
+#pragma unroll
+            for (int i = 0; i < 4; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
             // one ldmatrix brings the warp's eight keys for two k-steps
             const uint32_t bk = kb + (uint32_t)((buf * DT + warp * 8 + (lane & 7)) * ldk + 16 * (lane >> 3));
+#pragma unroll 2
             for (int ks = 0; ks < row16 / 16; ks += 2) {
                 uint32_t b[4], ah[4], al[4];
-                ldsm4(bk + 32 * ks, b);  // (an odd last k-step reads the zero padding column group or the next row; unused)
+                ldsm4(bk + 32 * ks, b);  // (an odd last k-step reads past its columns; unused)
                 ldsm4(qb + a_off + 32 * ks, ah);
                 ldsm4(qb + 16 * ldk + a_off + 32 * ks, al);
                 mma_bf16(s[0], ah, b[0], b[1]);
@@ -330,14 +341,16 @@ latent_decode_kernel(const float *__restrict__ qa, const bf16 *__restrict__ q, c
                 if (ks + 1 < row16 / 16) {
                     ldsm4(qb + a_off + 32 * ks + 32, ah);
                     ldsm4(qb + 16 * ldk + a_off + 32 * ks + 32, al);
-                    mma_bf16(s[0], ah, b[2], b[3]);
-                    mma_bf16(s[1], al, b[2], b[3]);
+                    mma_bf16(s[2], ah, b[2], b[3]);
+                    mma_bf16(s[3], al, b[2], b[3]);
                 }
             }
+#pragma unroll
+            for (int i = 0; i < 4; ++i) s[0][i] = (s[0][i] + s[2][i]) + (s[1][i] + s[3][i]);
             const int key = warp * 8 + 2 * tg;
             const bool i0 = t * DT + key < n, i1 = t * DT + key + 1 < n;
-            sc[g * 66 + key] = i0 ? (s[0][0] + s[1][0]) * scale : -INFINITY, sc[g * 66 + key + 1] = i1 ? (s[0][1] + s[1][1]) * scale : -INFINITY;
-            sc[(g + 8) * 66 + key] = i0 ? (s[0][2] + s[1][2]) * scale : -INFINITY, sc[(g + 8) * 66 + key + 1] = i1 ? (s[0][3] + s[1][3]) * scale : -INFINITY;
+            sc[g * 66 + key] = i0 ? s[0][0] * scale : -INFINITY, sc[g * 66 + key + 1] = i1 ? s[0][1] * scale : -INFINITY;
+            sc[(g + 8) * 66 + key] = i0 ? s[0][2] * scale : -INFINITY, sc[(g + 8) * 66 + key + 1] = i1 ? s[0][3] * scale : -INFINITY;
         }
         __syncthreads();
         // ---- running softmax: two heads per warp
@@ -405,7 +418,7 @@ latent_decode_kernel(const float *__restrict__ qa, const bf16 *__restrict__ q, c
     };
     if (threadIdx.x < DCL * 16) {
         const int k = threadIdx.x >> 4, hh = threadIdx.x & 15;
-        all_m[k][hh] = remote(&row_m[hh], k), all_l[k][hh] = remote(&row_l[hh], k);
+        all_m[k][hh] = k < cl ? remote(&row_m[hh], k) : -INFINITY, all_l[k][hh] = k < cl ? remote(&row_l[hh], k) : 0.f;
     }
     __syncthreads();
     if (threadIdx.x < 16) {
@@ -421,13 +434,13 @@ latent_decode_kernel(const float *__restrict__ qa, const bf16 *__restrict__ q, c
         for (int k = 0; k < DCL; ++k) all_f[k][hh] = __fdiv_rn(all_f[k][hh], den);
     }
     __syncthreads();
-    const int per = (rk + DCL - 1) / DCL, c0 = rank * per, c1 = min(rk, c0 + per);
+    const int per = (rk + cl - 1) / cl, c0 = rank * per, c1 = min(rk, c0 + per);
     for (int e = threadIdx.x; e < nh * per; e += 256) {
         const int hh = e / per, c = c0 + e % per;
         if (c >= c1) continue;
         float x[DCL], v = 0.f;
 #pragma unroll
-        for (int k = 0; k < DCL; ++k) x[k] = remote(&part[hh * ldp + c], k);  // zeros from a CTA without a tile, its factor is zero too
+        for (int k = 0; k < DCL; ++k) x[k] = k < cl ? remote(&part[hh * ldp + c], k) : 0.f;  // zeros from a CTA without a tile, its factor is zero too
 #pragma unroll
         for (int k = 0; k < DCL; ++k) v = fmaf(all_f[k][hh], x[k], v);
         oc[((size_t)r * heads + h0 + hh) * rk + c] = __float2bfloat16_rn(v);
@@ -642,10 +655,15 @@ int attend_absorbed_mma(smc_ctx *ctx, const smc_latent_dims &d, const smc_latent
     int rc = smc_launch_dense_grouped(ctx, b.q, d.heads * (d.dim + d.rot_dim), d.dim + d.rot_dim, b.w_ukt, d.heads, d.kv_rank, d.dim, rw.n, o, s);
     if (rc) return rc;
     const size_t smem = decode_smem(d);
+    // as many CTAs per row as keep the device full, up to the cluster limit and to one key tile each
+    int cl = DCL;
+    const int groups = (d.heads + 15) / 16, most = ((d.window > 0 ? d.window : max_seq) + DT - 1) / DT;
+    while (cl > 1 && ((long long)rw.n * groups * cl > ctx->sm_count || cl / 2 >= most)) cl /= 2;
     auto go = [&](auto kernel) {
         SMC_CUDA(ctx, cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-        smc_launch_dep(ctx->use_pdl, kernel, dim3(DCL, (d.heads + 15) / 16, rw.n), dim3(256), smem, s, (const float *)b.qa, (const bf16 *)b.q,
-                       (const bf16 *)b.cache, (bf16 *)b.oc, rw, sink, cosT, sinT, d.heads, d.dim, d.kv_rank, d.rot_dim, d.ring, d.window, d.scale, max_seq);
+        smc_launch_dep_cluster(ctx->use_pdl, cl, kernel, dim3(cl, groups, rw.n), dim3(256), smem, s, (const float *)b.qa, (const bf16 *)b.q,
+                               (const bf16 *)b.cache, (bf16 *)b.oc, rw, sink, cosT, sinT, d.heads, d.dim, d.kv_rank, d.rot_dim, d.ring, d.window, d.scale,
+                               max_seq);
         SMC_LAUNCH_CHECK(ctx);
         return (int)SMC_OK;
     };

@@ -25,32 +25,103 @@ __device__ __forceinline__ float silu(float z) { return __fdiv_rn(z, 1.0f + expf
 __device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
 // ------------------------------------------------------------------------------ convolution
-// A thread per channel walks CR rows.  Inputs before the portion come from the ring; those before position 0 are zero.
-// One row per sequence (decoding): the same launch stores the row's input, whose ring place nobody reads any more.
-constexpr int CR = 8;
-template <typename T>
-__global__ void __launch_bounds__(128) ssm_conv_kernel(const T *__restrict__ zx, int ld, int inner, T *__restrict__ out, T *__restrict__ ring, smc_rows rw,
-                                                       const float *__restrict__ w, const float *__restrict__ b, int ch, int taps)
+// A thread walks CR rows of V neighbouring channels, the last taps inputs in registers (TAPS = 0: taps read again for every
+// row, any number of them).  Inputs before the portion come from the ring; those before position 0 are zero.  One row per
+// sequence (decoding): the same launch stores the row's input, whose ring place nobody reads any more.
+template <typename T, int V> struct Pack;
+template <> struct Pack<float, 1> { using type = float; };
+template <> struct Pack<bf16, 1> { using type = bf16; };
+template <> struct Pack<bf16, 4> { using type = uint2; };
+template <> struct Pack<float, 4> { using type = float4; };
+template <typename T, int V>
+__device__ __forceinline__ void load_v(const T *p, float (&v)[V])
 {
-    smc_grid_dep_sync();
-    const int c = blockIdx.x * 128 + threadIdx.x;
-    if (c >= ch) return;
-    const int r0 = blockIdx.y * (rw.seq0 >= 0 ? CR : 1), r1 = min(rw.n, r0 + (rw.seq0 >= 0 ? CR : 1));
-    const int slot = rw.seq0 >= 0 ? rw.seq0 : r0, p0 = rw.pos[slot] - (rw.seq0 >= 0 ? 0 : r0);  // row r is at position p0 + r
-    T *rg = ring + (size_t)slot * taps * ch + c;
-    const float *wc = w + (size_t)c * taps;
-    const float bias = b[c];
-    for (int r = r0; r < r1; ++r) {
-        const int p = p0 + r, first = rw.seq0 >= 0 ? 0 : r;  // rows before `first` belong to other sequences
-        float acc = bias;
-        for (int j = taps - 1; j >= 0; --j) {  // oldest first
-            if (p - j < 0) continue;
-            const T v = r - j >= first ? zx[(size_t)(r - j) * ld + inner + c] : rg[(size_t)((p - j) % taps) * ch];
-            acc = fmaf(wc[taps - 1 - j], to_f(v), acc);
+    typename Pack<T, V>::type raw = *reinterpret_cast<const typename Pack<T, V>::type *>(p);
+    const T *e = reinterpret_cast<const T *>(&raw);
+#pragma unroll
+    for (int i = 0; i < V; ++i) v[i] = to_f(e[i]);
+}
+template <typename T, int V>
+__device__ __forceinline__ void store_v(T *p, const float (&v)[V])
+{
+    typename Pack<T, V>::type raw;
+    T *e = reinterpret_cast<T *>(&raw);
+#pragma unroll
+    for (int i = 0; i < V; ++i) e[i] = from_f<T>(v[i]);
+    *reinterpret_cast<typename Pack<T, V>::type *>(p) = raw;
+}
+// SiLU in front of a bfloat16 rounding may use the approximate exponential and quotient
+template <typename T> __device__ __forceinline__ float silu_for(float z) { return silu(z); }
+template <> __device__ __forceinline__ float silu_for<bf16>(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
+
+constexpr int CR = 16;
+template <typename T, int V, int TAPS>
+__global__ void __launch_bounds__(128) ssm_conv_kernel(const T *__restrict__ zx, int ld, int inner, T *__restrict__ out, T *__restrict__ ring, smc_rows rw,
+                                                       const float *__restrict__ w, const float *__restrict__ b, int ch, int ntaps)
+{
+    const int taps = TAPS ? TAPS : ntaps;
+    const int c = (blockIdx.x * 128 + threadIdx.x) * V;
+    const bool seq = rw.seq0 >= 0;
+    float wc[V][TAPS ? TAPS : 1], bias[V];
+    if (c < ch) {
+#pragma unroll
+        for (int i = 0; i < V; ++i) {
+            bias[i] = b[c + i];
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) wc[i][j] = w[(size_t)(c + i) * taps + j];
         }
-        out[(size_t)r * ch + c] = from_f<T>(silu(acc));
-        if (rw.seq0 < 0 || rw.n == 1) rg[(size_t)(p % taps) * ch] = zx[(size_t)r * ld + inner + c];
     }
+    smc_grid_dep_sync();
+    if (c >= ch) return;
+    const int r0 = blockIdx.y * (seq ? CR : 1), r1 = min(rw.n, r0 + (seq ? CR : 1)), first = seq ? 0 : r0;  // rows before `first` are other sequences'
+    const int slot = seq ? rw.seq0 : r0, p0 = rw.pos[slot] - (seq ? 0 : r0);                                 // row r is at position p0 + r
+    T *rg = ring + (size_t)slot * taps * ch + c;
+    auto input = [&](int r, float (&v)[V]) {
+#pragma unroll
+        for (int i = 0; i < V; ++i) v[i] = 0.f;
+        if (p0 + r < 0) return;
+        if (r >= first) load_v<T, V>(zx + (size_t)r * ld + inner + c, v);
+        else load_v<T, V>(rg + (size_t)((p0 + r) % taps) * ch, v);
+    };
+    if (TAPS) {
+        float hist[TAPS ? TAPS : 1][V];  // hist[j]: input of row r - taps + 1 + j
+#pragma unroll
+        for (int j = 0; j < TAPS - 1; ++j) input(r0 - TAPS + 1 + j, hist[j + 1]);
+#pragma unroll 4
+        for (int r = r0; r < r1; ++r) {
+#pragma unroll
+            for (int j = 0; j < TAPS - 1; ++j)
+#pragma unroll
+                for (int i = 0; i < V; ++i) hist[j][i] = hist[j + 1][i];
+            input(r, hist[TAPS - 1]);
+            float v[V];
+#pragma unroll
+            for (int i = 0; i < V; ++i) {
+                v[i] = bias[i];
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) v[i] = fmaf(wc[i][j], hist[j][i], v[i]);
+                v[i] = silu_for<T>(v[i]);
+            }
+            store_v<T, V>(out + (size_t)r * ch + c, v);
+        }
+    } else {
+        for (int r = r0; r < r1; ++r) {
+            float v[V], x[V];
+#pragma unroll
+            for (int i = 0; i < V; ++i) v[i] = bias[i];
+            for (int j = 0; j < taps; ++j) {
+                input(r - taps + 1 + j, x);
+#pragma unroll
+                for (int i = 0; i < V; ++i) v[i] = fmaf(w[(size_t)(c + i) * taps + j], x[i], v[i]);
+            }
+#pragma unroll
+            for (int i = 0; i < V; ++i) v[i] = silu_for<T>(v[i]);
+            store_v<T, V>(out + (size_t)r * ch + c, v);
+        }
+    }
+    if (!seq || rw.n == 1)
+        *reinterpret_cast<typename Pack<T, V>::type *>(rg + (size_t)((p0 + r0) % taps) * ch) =
+            *reinterpret_cast<const typename Pack<T, V>::type *>(zx + (size_t)r0 * ld + inner + c);
 }
 
 // The last `taps` inputs of a portion of several rows, after every reader of the old ones is done.
@@ -161,7 +232,15 @@ __device__ __forceinline__ void split2(float a, float b, uint32_t &hi, uint32_t 
     hi = *reinterpret_cast<const uint32_t *>(&h), lo = *reinterpret_cast<const uint32_t *>(&l);
 }
 
-constexpr int CQ = 64, CP = 32;
+// 2^x for x <= 0
+__device__ __forceinline__ float ex2(float x)
+{
+    float v;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(v) : "f"(x));
+    return v;
+}
+
+constexpr int CQ = 64, CP = 32, CTH = 512;
 struct ChunkSmem {  // byte offsets; rows are padded to an odd number of 16-byte units
     int ldn, cb, x, m, xw, st, f, total;
 };
@@ -175,13 +254,14 @@ __host__ __device__ inline ChunkSmem chunk_smem(int N)
     o.m = o.x + 2 * CQ * 80;                    // weights hi, lo [64][64]
     o.xw = o.m + 2 * CQ * 144;                  // scaled x hi, lo [64][32]
     o.st = o.xw + 2 * CQ * 80;                  // state hi, lo [32][N]
-    o.f = o.st + 2 * CP * o.ldn;                // dt, c, exp(c) [64] fp32 each, then exp(c_end)
-    o.total = o.f + 3 * CQ * 4 + 16;
+    o.f = o.st + 2 * CP * o.ldn + 32;           // two buffers of dt, c, 2^c, 2^(c_end - c) dt [64] fp32 each, then 2^c_end
+    o.total = o.f + 2 * (4 * CQ + 4) * 4;
     return o;
 }
 
-template <int NTW>  // state tiles of 8 columns per warp (four warps across N)
-__global__ void __launch_bounds__(256) ssm_chunk_kernel(const bf16 *__restrict__ xbc, const float *__restrict__ dt_raw, float *__restrict__ y,
+// 16 warps: token tile warp % 4 against a quarter of the other side.
+template <int NTW>  // state tiles of 8 columns per warp (eight warps across N)
+__global__ void __launch_bounds__(CTH) ssm_chunk_kernel(const bf16 *__restrict__ xbc, const float *__restrict__ dt_raw, float *__restrict__ y,
                                                         float *__restrict__ state, smc_rows rw, const float *__restrict__ dt_bias,
                                                         const float *__restrict__ a_log, const float *__restrict__ d_skip, int heads, int P, int N,
                                                         int groups)
@@ -191,17 +271,17 @@ __global__ void __launch_bounds__(256) ssm_chunk_kernel(const bf16 *__restrict__
     const uint32_t sb = (uint32_t)__cvta_generic_to_shared(csm);
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, tg = lane & 3;
     const int h = blockIdx.x, p0 = blockIdx.y * CP, grp = h / (heads / groups), T = rw.n;
-    const int inner = heads * P, ch = inner + 2 * groups * N, n16 = (N + 15) & ~15;
-    float *s_dt = reinterpret_cast<float *>(csm + L.f), *s_c = s_dt + CQ, *s_ec = s_c + CQ, *s_end = s_ec + CQ;
-    for (int e = threadIdx.x; e < L.total / 16; e += 256) reinterpret_cast<uint4 *>(csm)[e] = make_uint4(0u, 0u, 0u, 0u);
+    const int inner = heads * P, ch = inner + 2 * groups * N, n16 = (N + 15) & ~15, ksteps = n16 / 16;
+    for (int e = threadIdx.x; e < L.total / 16; e += CTH) reinterpret_cast<uint4 *>(csm)[e] = make_uint4(0u, 0u, 0u, 0u);
     smc_grid_dep_sync();
     __syncthreads();
     const bool fresh = rw.pos[rw.seq0] == 0;
     float *st = state + ((size_t)rw.seq0 * heads + h) * P * N;
-    const float A = -expf(a_log[h]), D = d_skip[h], bias = dt_bias[h];
+    const float D = d_skip[h], bias = dt_bias[h];
+    const double A2 = -(double)expf(a_log[h]) * 1.4426950408889634;  // log decays are kept as powers of two
     const int cn = N / 8, cx = min(CP, P - p0) / 8, per = 2 * cn + cx;
     auto fetch = [&](int t0, int buf) {
-        for (int e = threadIdx.x; e < CQ * per; e += 256) {
+        for (int e = threadIdx.x; e < CQ * per; e += CTH) {
             const int t = e / per, c = e % per;
             const bool in = t0 + t < T;
             const bf16 *src = xbc + (size_t)(in ? t0 + t : T - 1) * ch;
@@ -211,11 +291,36 @@ __global__ void __launch_bounds__(256) ssm_chunk_kernel(const bf16 *__restrict__
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
+    // step sizes and running log decays of a chunk by one warp, two tokens per lane; past the end: no input, no decay
+    float raw0 = 0.f, raw1 = 0.f;
+    auto load_dt = [&](int t0) {
+        const int t = t0 + 2 * lane;
+        raw0 = t < T ? dt_raw[(size_t)t * heads + h] : 0.f, raw1 = t + 1 < T ? dt_raw[(size_t)(t + 1) * heads + h] : 0.f;
+    };
+    auto prepare = [&](int t0, int buf) {
+        float *f = reinterpret_cast<float *>(csm + L.f) + buf * (4 * CQ + 4);
+        const int t = t0 + 2 * lane;
+        const float d0 = t < T ? softplus(raw0 + bias) : 0.f, d1 = t + 1 < T ? softplus(raw1 + bias) : 0.f;
+        const double a1 = A2 * d1;
+        double sum = A2 * d0 + a1;
+        for (int d = 1; d < 32; d <<= 1) {
+            const double v = __shfl_up_sync(0xffffffffu, sum, d);
+            if (lane >= d) sum += v;
+        }
+        const double end = __shfl_sync(0xffffffffu, sum, 31);
+        const float c0 = (float)(sum - a1), c1 = (float)sum;
+        *reinterpret_cast<float2 *>(f + 2 * lane) = make_float2(d0, d1);
+        *reinterpret_cast<float2 *>(f + CQ + 2 * lane) = make_float2(c0, c1);
+        *reinterpret_cast<float2 *>(f + 2 * CQ + 2 * lane) = make_float2(ex2(c0), ex2(c1));
+        *reinterpret_cast<float2 *>(f + 3 * CQ + 2 * lane) = make_float2(ex2((float)(end - (sum - a1))) * d0, ex2((float)(end - sum)) * d1);
+        if (lane == 0) f[4 * CQ] = ex2((float)end);
+    };
     fetch(0, 0);
-    // state accumulators: rows p (16 per warp pair member), columns n
-    const int sm_m = warp & 1, sm_n = warp >> 1;  // 16-row tile of the 32 columns of x, quarter of N
+    if (warp == 0) load_dt(0), prepare(0, 0);
+    // state accumulators: rows p (two tiles of 16), columns n (an eighth each)
+    const int sm_m = warp & 1, sm_n = warp >> 1;
     float S[NTW][4];
-    const int nt_per = (n16 / 8 + 3) / 4;
+    const int nt_per = (n16 / 8 + 7) / 8;
 #pragma unroll
     for (int i = 0; i < NTW; ++i) {
         S[i][0] = S[i][1] = S[i][2] = S[i][3] = 0.f;
@@ -242,120 +347,108 @@ __global__ void __launch_bounds__(256) ssm_chunk_kernel(const bf16 *__restrict__
     // ldmatrix lane offsets: A operand rows / B operand [n][k] rows, two tiles / transposed [k][n]
     const int la = (lane & 7) + 8 * ((lane >> 3) & 1), lah = 16 * (lane >> 4);
     const int lb = (lane & 7) + 8 * (lane >> 4), lbh = 16 * ((lane >> 3) & 1);
-    const int mt = warp & 3, nh = warp >> 2;      // 16-token tile, half of the other side
+    const int mt = warp & 3, nq = warp >> 2;
     int buf = 0;
     for (int t0 = 0; t0 < T; t0 += CQ, buf ^= 1) {
-        if (t0 + CQ < T) {
+        const bool more = t0 + CQ < T;
+        if (more) {
             fetch(t0 + CQ, buf ^ 1);
+            if (warp == 0) load_dt(t0 + CQ);
             asm volatile("cp.async.wait_group 1;" ::: "memory");
         } else {
             asm volatile("cp.async.wait_group 0;" ::: "memory");
         }
-        if (warp == 0) {  // step sizes and running log decays of the chunk: two tokens per lane
-            float dt[2];
-            double a[2];
-#pragma unroll
-            for (int i = 0; i < 2; ++i) {
-                const int t = t0 + 2 * lane + i;
-                dt[i] = t < T ? softplus(dt_raw[(size_t)t * heads + h] + bias) : 0.f;  // past the end: no input, no decay
-                a[i] = (double)(A * dt[i]);
-            }
-            double sum = a[0] + a[1];
-            for (int d = 1; d < 32; d <<= 1) {
-                const double v = __shfl_up_sync(0xffffffffu, sum, d);
-                if (lane >= d) sum += v;
-            }
-            const float c0 = (float)(sum - a[1]), c1 = (float)sum;
-            s_dt[2 * lane] = dt[0], s_dt[2 * lane + 1] = dt[1];
-            s_c[2 * lane] = c0, s_c[2 * lane + 1] = c1;
-            s_ec[2 * lane] = expf(c0), s_ec[2 * lane + 1] = expf(c1);
-            if (lane == 31) *s_end = c1;
-        }
         __syncthreads();
+        const float *s_dt = reinterpret_cast<const float *>(csm + L.f) + buf * (4 * CQ + 4), *s_c = s_dt + CQ, *s_ec = s_c + CQ, *s_w = s_ec + CQ;
         const uint32_t cC = sb + L.cb + (uint32_t)(2 * buf * CQ * L.ldn), cB = cC + (uint32_t)(CQ * L.ldn), cX = sb + L.x + (uint32_t)(buf * CQ * 80);
-        // ---- weights of the first sum: C_t . B_s for 16 tokens x 32 sources per warp
-        float G[4][4], Y[2][4];
+        // ---- C_t . B_s for 16 tokens x 16 sources, and S^T C for 16 tokens x 8 value columns
+        float G[2][4], Y[2][4];
 #pragma unroll
-        for (int i = 0; i < 4; ++i) G[i][0] = G[i][1] = G[i][2] = G[i][3] = 0.f;
+        for (int i = 0; i < 2; ++i) G[i][0] = G[i][1] = G[i][2] = G[i][3] = Y[i][0] = Y[i][1] = Y[i][2] = Y[i][3] = 0.f;
+        const bool any = nq <= mt;  // else every source lies after every token
+        for (int k = 0; k < ksteps; k += 2) {
+            uint32_t sh[4], sl[4];  // eight state rows for two k-steps (of an odd last pair only the first half is used)
+            ldsm4(sb + L.st + (uint32_t)((8 * nq + (lane & 7)) * L.ldn + 32 * k + 16 * (lane >> 3)), sh);
+            ldsm4(sb + L.st + (uint32_t)((CP + 8 * nq + (lane & 7)) * L.ldn + 32 * k + 16 * (lane >> 3)), sl);
 #pragma unroll
-        for (int i = 0; i < 2; ++i) Y[i][0] = Y[i][1] = Y[i][2] = Y[i][3] = 0.f;
-        const bool any = 32 * nh <= 16 * mt + 15;  // else every source lies after every token
-        for (int k = 0; k < n16 / 16; ++k) {
-            uint32_t a[4], b[4], sh[4], sl[4];
-            ldsm4(cC + (uint32_t)((16 * mt + la) * L.ldn + 32 * k + lah), a);
-            if (any) {
-#pragma unroll
-                for (int j = 0; j < 2; ++j) {
-                    ldsm4(cB + (uint32_t)((32 * nh + 16 * j + lb) * L.ldn + 32 * k + lbh), b);
-                    mma_bf16(G[2 * j], a, b[0], b[1]);
-                    mma_bf16(G[2 * j + 1], a, b[2], b[3]);
+            for (int j = 0; j < 2; ++j)
+                if (k + j < ksteps) {
+                    uint32_t a[4];
+                    ldsm4(cC + (uint32_t)((16 * mt + la) * L.ldn + 32 * (k + j) + lah), a);
+                    if (any) {
+                        uint32_t b[4];
+                        ldsm4(cB + (uint32_t)((16 * nq + lb) * L.ldn + 32 * (k + j) + lbh), b);
+                        mma_bf16(G[0], a, b[0], b[1]);
+                        mma_bf16(G[1], a, b[2], b[3]);
+                    }
+                    mma_bf16(Y[0], a, sl[2 * j], sl[2 * j + 1]);
+                    mma_bf16(Y[1], a, sh[2 * j], sh[2 * j + 1]);
                 }
-            }
-            // ---- S^T C: 16 tokens x 16 value columns per warp
-            ldsm4(sb + L.st + (uint32_t)((16 * nh + lb) * L.ldn + 32 * k + lbh), sh);
-            ldsm4(sb + L.st + (uint32_t)((CP + 16 * nh + lb) * L.ldn + 32 * k + lbh), sl);
-            mma_bf16(Y[0], a, sl[0], sl[1]), mma_bf16(Y[1], a, sl[2], sl[3]);
-            mma_bf16(Y[0], a, sh[0], sh[1]), mma_bf16(Y[1], a, sh[2], sh[3]);
         }
-        {
-            const int ta = 16 * mt + g, tb = ta + 8;
+        const int ta = 16 * mt + g, tb = ta + 8;
+        if (any) {
             const float ca = s_c[ta], cb = s_c[tb];
 #pragma unroll
-            for (int i = 0; i < 4; ++i) {
-                const int s = 32 * nh + 8 * i + 2 * tg;
-                float w[4];
-#pragma unroll
-                for (int j = 0; j < 2; ++j) {
-                    w[j] = s + j <= ta ? G[i][j] * (expf(ca - s_c[s + j]) * s_dt[s + j]) : 0.f;
-                    w[2 + j] = s + j <= tb ? G[i][2 + j] * (expf(cb - s_c[s + j]) * s_dt[s + j]) : 0.f;
-                }
+            for (int i = 0; i < 2; ++i) {
+                const int s = 16 * nq + 8 * i + 2 * tg;
+                const float2 cs = *reinterpret_cast<const float2 *>(s_c + s), ds = *reinterpret_cast<const float2 *>(s_dt + s);
+                // (a source after the token would have a growing factor: its exponent is clamped and its weight zeroed)
+                const float w0 = s <= ta ? G[i][0] * (ex2(fminf(ca - cs.x, 0.f)) * ds.x) : 0.f, w1 = s + 1 <= ta ? G[i][1] * (ex2(fminf(ca - cs.y, 0.f)) * ds.y) : 0.f;
+                const float w2 = s <= tb ? G[i][2] * (ex2(fminf(cb - cs.x, 0.f)) * ds.x) : 0.f, w3 = s + 1 <= tb ? G[i][3] * (ex2(fminf(cb - cs.y, 0.f)) * ds.y) : 0.f;
                 uint32_t hi, lo;
                 uint8_t *d = csm + L.m + ta * 144 + 2 * s;
-                split2(w[0], w[1], hi, lo);
+                split2(w0, w1, hi, lo);
                 *reinterpret_cast<uint32_t *>(d) = hi, *reinterpret_cast<uint32_t *>(d + CQ * 144) = lo;
-                split2(w[2], w[3], hi, lo);
+                split2(w2, w3, hi, lo);
                 d += 8 * 144;
                 *reinterpret_cast<uint32_t *>(d) = hi, *reinterpret_cast<uint32_t *>(d + CQ * 144) = lo;
             }
-            const float ea = s_ec[ta], eb = s_ec[tb];
-#pragma unroll
-            for (int i = 0; i < 2; ++i) Y[i][0] *= ea, Y[i][1] *= ea, Y[i][2] *= eb, Y[i][3] *= eb;
         }
+        const float ea = s_ec[ta], eb = s_ec[tb];
+        Y[0][0] = (Y[0][0] + Y[1][0]) * ea, Y[0][1] = (Y[0][1] + Y[1][1]) * ea, Y[0][2] = (Y[0][2] + Y[1][2]) * eb, Y[0][3] = (Y[0][3] + Y[1][3]) * eb;
+        Y[1][0] = Y[1][1] = Y[1][2] = Y[1][3] = 0.f;
         // ---- x scaled for the state update
-        const float end = *s_end;
-        for (int e = threadIdx.x; e < CQ * CP / 2; e += 256) {
+#pragma unroll
+        for (int e = threadIdx.x; e < CQ * CP / 2; e += CTH) {
             const int t = e >> 4, c = (e & 15) * 2;
-            const float f = expf(end - s_c[t]) * s_dt[t];
+            const float f = s_w[t];
             const __nv_bfloat162 v = *reinterpret_cast<const __nv_bfloat162 *>(csm + L.x + (buf * CQ + t) * 80 + 2 * c);
             uint32_t hi, lo;
             split2(__bfloat162float(v.x) * f, __bfloat162float(v.y) * f, hi, lo);
             *reinterpret_cast<uint32_t *>(csm + L.xw + t * 80 + 2 * c) = hi, *reinterpret_cast<uint32_t *>(csm + L.xw + (CQ + t) * 80 + 2 * c) = lo;
         }
         __syncthreads();
-        // ---- y: weights x x, sources up to the tile's last token
-        for (int k = 0; k <= mt; ++k) {
-            uint32_t ah[4], al[4], b[4];
-            ldsm4(sb + L.m + (uint32_t)((16 * mt + la) * 144 + 32 * k + lah), ah);
-            ldsm4(sb + L.m + (uint32_t)((CQ + 16 * mt + la) * 144 + 32 * k + lah), al);
-            ldsm4t(cX + (uint32_t)((16 * k + la) * 80 + 32 * nh + lah), b);
-            mma_bf16(Y[0], al, b[0], b[1]), mma_bf16(Y[1], al, b[2], b[3]);
-            mma_bf16(Y[0], ah, b[0], b[1]), mma_bf16(Y[1], ah, b[2], b[3]);
+        // ---- y: weights times x, sources up to the tile's last token (weights past it were never written: stay below)
+#pragma unroll
+        for (int k = 0; k < CQ / 16; k += 2) {
+            if (k > mt) break;
+            uint32_t b[4];  // eight value columns for 32 sources
+            ldsm4t(cX + (uint32_t)((16 * k + lane) * 80 + 16 * nq), b);
+#pragma unroll
+            for (int j = 0; j < 2; ++j)
+                if (k + j <= mt) {
+                    uint32_t ah[4], al[4];
+                    ldsm4(sb + L.m + (uint32_t)((16 * mt + la) * 144 + 32 * (k + j) + lah), ah);
+                    ldsm4(sb + L.m + (uint32_t)((CQ + 16 * mt + la) * 144 + 32 * (k + j) + lah), al);
+                    mma_bf16(Y[1], al, b[2 * j], b[2 * j + 1]);
+                    mma_bf16(Y[0], ah, b[2 * j], b[2 * j + 1]);
+                }
         }
+        {
+            const int c = 8 * nq + 2 * tg;
+            if (p0 + c < P) {
 #pragma unroll
-        for (int i = 0; i < 2; ++i) {
-            const int c = 16 * nh + 8 * i + 2 * tg;
-            if (p0 + c >= P) continue;
-#pragma unroll
-            for (int j = 0; j < 2; ++j) {
-                const int t = 16 * mt + g + 8 * j;
-                if (t0 + t >= T) continue;
-                const __nv_bfloat162 v = *reinterpret_cast<const __nv_bfloat162 *>(csm + L.x + (buf * CQ + t) * 80 + 2 * c);
-                *reinterpret_cast<float2 *>(y + (size_t)(t0 + t) * inner + h * P + p0 + c) =
-                    make_float2(fmaf(D, __bfloat162float(v.x), Y[i][2 * j]), fmaf(D, __bfloat162float(v.y), Y[i][2 * j + 1]));
+                for (int j = 0; j < 2; ++j) {
+                    const int t = ta + 8 * j;
+                    if (t0 + t >= T) continue;
+                    const __nv_bfloat162 v = *reinterpret_cast<const __nv_bfloat162 *>(csm + L.x + (buf * CQ + t) * 80 + 2 * c);
+                    *reinterpret_cast<float2 *>(y + (size_t)(t0 + t) * inner + h * P + p0 + c) =
+                        make_float2(fmaf(D, __bfloat162float(v.x), Y[0][2 * j] + Y[1][2 * j]), fmaf(D, __bfloat162float(v.y), Y[0][2 * j + 1] + Y[1][2 * j + 1]));
+                }
             }
         }
         // ---- state
-        const float dec = expf(end);
+        const float dec = s_dt[4 * CQ];
 #pragma unroll
         for (int i = 0; i < NTW; ++i) S[i][0] *= dec, S[i][1] *= dec, S[i][2] *= dec, S[i][3] *= dec;
 #pragma unroll
@@ -370,12 +463,13 @@ __global__ void __launch_bounds__(256) ssm_chunk_kernel(const bf16 *__restrict__
                 const int nt = sm_n * nt_per + i;
                 if (i >= nt_per || nt * 8 >= n16) continue;
                 uint32_t b[4];
-                // two tiles; the second may lie past this warp's share: its product is then not used
+                // two tiles; where the second lies past the row's end the first is read twice, where it is another warp's it is not used
                 ldsm4t(cB + (uint32_t)((16 * k + la) * L.ldn + 16 * nt + (nt * 8 + 8 < n16 ? lah : 0)), b);
                 mma_bf16(S[i], al, b[0], b[1]), mma_bf16(S[i], ah, b[0], b[1]);
                 if (i + 1 < nt_per) mma_bf16(S[i + 1], al, b[2], b[3]), mma_bf16(S[i + 1], ah, b[2], b[3]);
             }
         }
+        if (warp == 0 && more) prepare(t0 + CQ, buf ^ 1);  // this warp has the least of the triangle above
         __syncthreads();  // everybody has read the state planes, the weights and this chunk's buffers
         put_state();
     }
@@ -389,26 +483,36 @@ __global__ void __launch_bounds__(256) ssm_chunk_kernel(const bf16 *__restrict__
 }
 
 // ------------------------------------------------------------------------------ gate, then norm in parts
-template <typename T>
+template <typename T, int V>
 __global__ void __launch_bounds__(128) ssm_gate_norm_kernel(const float *__restrict__ y, const T *__restrict__ zx, int ld, const float *__restrict__ w,
                                                             T *__restrict__ o, int inner, int parts, float eps)
 {
-    extern __shared__ float sv[];
+    extern __shared__ __align__(16) float sv[];
     __shared__ float red[4];
     smc_grid_dep_sync();
     const int n = inner / parts, r = blockIdx.x, base = blockIdx.y * n;
     float ss = 0.f;
-    for (int i = threadIdx.x; i < n; i += 128) {
-        const float v = y[(size_t)r * inner + base + i] * silu(to_f(zx[(size_t)r * ld + base + i]));
-        sv[i] = v;
-        ss = fmaf(v, v, ss);
+    for (int i = threadIdx.x * V; i < n; i += 128 * V) {
+        float a[V], z[V];
+        load_v<float, V>(y + (size_t)r * inner + base + i, a);
+        load_v<T, V>(zx + (size_t)r * ld + base + i, z);
+#pragma unroll
+        for (int j = 0; j < V; ++j) a[j] *= silu_for<T>(z[j]), ss = fmaf(a[j], a[j], ss);
+        store_v<float, V>(sv + i, a);
     }
     ss = smc_group_sum<32>(ss);
     if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
     __syncthreads();
     ss = (red[0] + red[1]) + (red[2] + red[3]);
     const float inv = __fdiv_rn(1.0f, sqrtf(__fdiv_rn(ss, (float)n) + eps));
-    for (int i = threadIdx.x; i < n; i += 128) o[(size_t)r * inner + base + i] = from_f<T>((sv[i] * inv) * w[base + i]);
+    for (int i = threadIdx.x * V; i < n; i += 128 * V) {
+        float a[V], g[V];
+        load_v<float, V>(sv + i, a);
+        load_v<float, V>(w + base + i, g);
+#pragma unroll
+        for (int j = 0; j < V; ++j) a[j] = (a[j] * inv) * g[j];
+        store_v<T, V>(o + (size_t)r * inner + base + i, a);
+    }
 }
 
 // portions from this many rows on are taken in chunks
@@ -423,14 +527,12 @@ int recur_chunks(smc_ctx *ctx, const smc_ssm_dims &d, const smc_ssm_bufs &b, con
     if (d.vdim % 8 || d.state % 8 || d.state > 256 || L.total > 220 * 1024) return SMC_E_UNSUPPORTED;
     auto go = [&](auto kernel) {
         SMC_CUDA(ctx, cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, L.total));
-        smc_launch_dep(ctx->use_pdl, kernel, dim3(d.heads, (d.vdim + CP - 1) / CP), dim3(256), (size_t)L.total, s, (const bf16 *)b.xbc, b.dt_raw, b.y,
+        smc_launch_dep(ctx->use_pdl, kernel, dim3(d.heads, (d.vdim + CP - 1) / CP), dim3(CTH), (size_t)L.total, s, (const bf16 *)b.xbc, b.dt_raw, b.y,
                        b.state, rw, dt_bias, a_log, d_skip, d.heads, d.vdim, d.state, d.groups);
         SMC_LAUNCH_CHECK(ctx);
         return (int)SMC_OK;
     };
-    if (d.state <= 64) return go(ssm_chunk_kernel<2>);
-    if (d.state <= 128) return go(ssm_chunk_kernel<4>);
-    return go(ssm_chunk_kernel<8>);
+    return d.state <= 128 ? go(ssm_chunk_kernel<2>) : go(ssm_chunk_kernel<4>);
 }
 
 template <typename T>
@@ -463,8 +565,15 @@ int mix(smc_ctx *ctx, const smc_ssm_dims &d, const smc_ssm_bufs &b, const smc_ro
 {
     const int inner = d.heads * d.vdim, ch = inner + 2 * d.groups * d.state;
     const bool seq = rw.seq0 >= 0;
-    smc_launch_dep(ctx->use_pdl, ssm_conv_kernel<T>, dim3((ch + 127) / 128, seq ? (rw.n + CR - 1) / CR : rw.n), dim3(128), 0, s,
-                   static_cast<const T *>(b.zx), b.ld, inner, static_cast<T *>(b.xbc), static_cast<T *>(b.conv_state), rw, conv_w, conv_b, ch, d.conv);
+    auto conv = [&](auto kernel, int v) {
+        smc_launch_dep(ctx->use_pdl, kernel, dim3((ch / v + 127) / 128, seq ? (rw.n + CR - 1) / CR : rw.n), dim3(128), 0, s, static_cast<const T *>(b.zx),
+                       b.ld, inner, static_cast<T *>(b.xbc), static_cast<T *>(b.conv_state), rw, conv_w, conv_b, ch, d.conv);
+    };
+    const bool four = inner % 4 == 0 && ch % 4 == 0 && b.ld % 4 == 0;
+    if (d.conv == 4) four ? conv(ssm_conv_kernel<T, 4, 4>, 4) : conv(ssm_conv_kernel<T, 1, 4>, 1);
+    else if (d.conv == 3) four ? conv(ssm_conv_kernel<T, 4, 3>, 4) : conv(ssm_conv_kernel<T, 1, 3>, 1);
+    else if (d.conv == 2) four ? conv(ssm_conv_kernel<T, 4, 2>, 4) : conv(ssm_conv_kernel<T, 1, 2>, 1);
+    else four ? conv(ssm_conv_kernel<T, 4, 0>, 4) : conv(ssm_conv_kernel<T, 1, 0>, 1);
     SMC_LAUNCH_CHECK(ctx);
     if (seq && rw.n > 1) {
         smc_launch_dep(ctx->use_pdl, ssm_conv_keep_kernel<T>, dim3((ch + 127) / 128, d.conv < rw.n ? d.conv : rw.n), dim3(128), 0, s,
@@ -475,9 +584,13 @@ int mix(smc_ctx *ctx, const smc_ssm_dims &d, const smc_ssm_bufs &b, const smc_ro
     if (rc == SMC_E_UNSUPPORTED) rc = recur_steps<T>(ctx, d, b, rw, dt_bias, a_log, d_skip, s);
     if (rc) return rc;
     const size_t nsm = (size_t)(inner / d.norm_groups) * sizeof(float);
-    if (nsm > 40 * 1024) SMC_CUDA(ctx, cudaFuncSetAttribute(ssm_gate_norm_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)nsm));
-    smc_launch_dep(ctx->use_pdl, ssm_gate_norm_kernel<T>, dim3(rw.n, d.norm_groups), dim3(128), nsm, s, (const float *)b.y, static_cast<const T *>(b.zx),
-                   b.ld, norm, static_cast<T *>(b.o), inner, d.norm_groups, d.eps);
+    auto gate = [&](auto kernel) {
+        if (nsm > 40 * 1024) cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)nsm);
+        smc_launch_dep(ctx->use_pdl, kernel, dim3(rw.n, d.norm_groups), dim3(128), nsm, s, (const float *)b.y, static_cast<const T *>(b.zx), b.ld, norm,
+                       static_cast<T *>(b.o), inner, d.norm_groups, d.eps);
+    };
+    if (inner / d.norm_groups % 4 == 0 && b.ld % 4 == 0) gate(ssm_gate_norm_kernel<T, 4>);
+    else gate(ssm_gate_norm_kernel<T, 1>);
     SMC_LAUNCH_CHECK(ctx);
     return SMC_OK;
 }
