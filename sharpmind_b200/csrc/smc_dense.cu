@@ -448,9 +448,10 @@ int smc_launch_dense_rows(smc_ctx *ctx, const void *x, int x_bf16, int ldx, cons
     if (vec) {
         const bf16 *xb = static_cast<const bf16 *>(x);
         if (M > 32 && aligned(o.y)) {
-            const int mt = (M + TC_M - 1) / TC_M;
-            // wide tiles once they fill the device, narrow ones for smaller products
-            if ((long long)mt * ((N + 255) / 256) >= ctx->sm_count) return launch_tc<256>(ctx, xb, ldx, w, M, N, K, o, s);
+            // rounds of tiles over the device: a wide tile takes less than twice as long as a narrow one
+            const long long mt = (M + TC_M - 1) / TC_M, sms = ctx->sm_count;
+            const long long wide = 2 * ((mt * ((N + 255) / 256) + sms - 1) / sms), narrow = (mt * ((N + 127) / 128) + sms - 1) / sms;
+            if (5 * wide <= 6 * narrow) return launch_tc<256>(ctx, xb, ldx, w, M, N, K, o, s);
             return launch_tc<128>(ctx, xb, ldx, w, M, N, K, o, s);
         }
         launch_skinny(ctx, xb, ldx, 0, w, 1, N, K, M, o, s);

@@ -242,6 +242,13 @@ __device__ __forceinline__ void cp16(uint32_t dst, const void *src, bool in)
 {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(in ? 16 : 0) : "memory");
 }
+// 2^x for x <= 0
+__device__ __forceinline__ float ex2(float x)
+{
+    float v;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(v) : "f"(x));
+    return v;
+}
 __device__ __forceinline__ uint32_t pack2(float a, float b)
 {
     const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
@@ -253,12 +260,16 @@ __device__ __forceinline__ uint32_t pack2(float a, float b)
 // the cluster merges its partial sums through distributed shared memory.  The absorbed query (fp32) enters as a bfloat16 pair hi + lo,
 // so scores keep 16 bits of it; the cached rows are exact operands of both products.  All heads read the same keys: a tile
 // is fetched once per 16 heads.
-//   shared memory: query planes [2][16][ldk], two key tiles [64][ldk], scores [16][66] fp32, weights [16][72] bfloat16
+// Scores split their sum over the latent across eight warps (twice, for the halves of a tile): a warp keeps its slice of the query in registers for all tiles and
+// reads its slice of every key once; the eight partial score tiles meet in shared memory.
+//   shared memory: query planes [2][16][ldk], later the partial scores [8][16][72] fp32; two key tiles [64][ldk]; weights
+//   [16][72] bfloat16
 // The keys and the position are fetched BEFORE the wait for the predecessor: they were written by the kernel before it, and a
 // kernel that is launched early is so only after every CTA of its predecessor has passed its own wait.
-constexpr int DT = 64, DCL = 8;
-template <int OPW>  // 16-column groups of the latent a warp accumulates (8 warps)
-__global__ void __launch_bounds__(256)
+constexpr int DT = 64, DCL = 8, KPW = 5, DTH = 512, DLS = 72;  // keys per tile, largest cluster, 16-element slices of the sum per warp, threads, score row
+__host__ __device__ inline int decode_head_bytes(int ldk) { return 2 * 16 * ldk > 8 * 16 * DLS * 4 ? 2 * 16 * ldk : 8 * 16 * DLS * 4; }
+template <int OPW>  // 16-column groups of the latent a warp accumulates (16 warps)
+__global__ void __launch_bounds__(DTH)
 latent_decode_kernel(const float *__restrict__ qa, const bf16 *__restrict__ q, const bf16 *__restrict__ cache, bf16 *__restrict__ oc, smc_rows rw,
                      const float *__restrict__ sink, const float *__restrict__ cosT, const float *__restrict__ sinT, int heads, int dim, int rk, int rd,
                      int ring, int window, float scale, int max_seq)
@@ -268,14 +279,17 @@ latent_decode_kernel(const float *__restrict__ qa, const bf16 *__restrict__ q, c
     const int row = rk + rd, row16 = (row + 15) & ~15, ldk = (row16 + 8) * 2;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, tg = lane & 3;
     const int rank = blockIdx.x, h0 = blockIdx.y * 16, nh = min(16, heads - h0), r = blockIdx.z;
-    uint8_t *q_s = sm_raw, *k_s = q_s + 2 * 16 * ldk, *s_s = k_s + 2 * DT * ldk, *p_s = s_s + 16 * 66 * 4;
+    uint8_t *q_s = sm_raw, *k_s = q_s + decode_head_bytes(ldk), *p_s = k_s + 2 * DT * ldk;
     const uint32_t qb = (uint32_t)__cvta_generic_to_shared(q_s), kb = (uint32_t)__cvta_generic_to_shared(k_s), pb = (uint32_t)__cvta_generic_to_shared(p_s);
-    float *sc = reinterpret_cast<float *>(s_s);
+    float *sc = reinterpret_cast<float *>(q_s);
     const int cl = gridDim.x;
     // padding columns of the planes and tiles, and the planes' rows without a head
     const int pad = ldk / 2 - row;
-    for (int e = threadIdx.x; e < (2 * 16 + 2 * DT) * pad; e += 256) reinterpret_cast<bf16 *>(sm_raw + (e / pad) * ldk)[row + e % pad] = __float2bfloat16_rn(0.f);
-    for (int e = threadIdx.x; e < 2 * (16 - nh) * row; e += 256) {
+    for (int e = threadIdx.x; e < (2 * 16 + 2 * DT) * pad; e += DTH) {
+        const int j = e / pad;
+        reinterpret_cast<bf16 *>(j < 32 ? q_s + j * ldk : k_s + (j - 32) * ldk)[row + e % pad] = __float2bfloat16_rn(0.f);
+    }
+    for (int e = threadIdx.x; e < 2 * (16 - nh) * row; e += DTH) {
         const int rr = e / row, pl = rr / (16 - nh);
         reinterpret_cast<bf16 *>(sm_raw + (pl * 16 + nh + rr % (16 - nh)) * ldk)[e % row] = __float2bfloat16_rn(0.f);
     }
@@ -283,12 +297,15 @@ latent_decode_kernel(const float *__restrict__ qa, const bf16 *__restrict__ q, c
     row_place(rw, r, slot, p);
     const int lo = window > 0 ? max(0, p - window + 1) : 0, n = p - lo + 1, tiles = (n + DT - 1) / DT;
     const bf16 *base = cache + (size_t)slot * ring * row;
-    const int chunks = row / 8;
-    auto fetch = [&](int t, int buf) {
-        for (int e = threadIdx.x; e < DT * chunks; e += 256) {
-            const int j = e / chunks, c = e % chunks, k = t * DT + j;
+    const int chunks = row / 8, lo_row = lo % ring;
+    auto fetch = [&](int t, int buf) {  // a warp per row
+        for (int j = warp; j < DT; j += DTH / 32) {
+            const int k = t * DT + j;
             const bool in = k < n;
-            cp16(kb + (uint32_t)((buf * DT + j) * ldk + 16 * c), base + (size_t)((lo + (in ? k : 0)) % ring) * row + 8 * c, in);
+            int rr = lo_row + (in ? k : 0);
+            rr -= rr >= ring ? ring : 0;  // n <= ring
+            const bf16 *src = base + (size_t)rr * row;
+            for (int c = lane; c < chunks; c += 32) cp16(kb + (uint32_t)((buf * DT + j) * ldk + 16 * c), src + 8 * c, in);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -299,9 +316,20 @@ latent_decode_kernel(const float *__restrict__ qa, const bf16 *__restrict__ q, c
         reinterpret_cast<bf16 *>(q_s + hh * ldk)[i] = hi;
         reinterpret_cast<bf16 *>(q_s + (16 + hh) * ldk)[i] = __float2bfloat16_rn(v - __bfloat162float(hi));
     };
-    for (int e = threadIdx.x; e < nh * rk; e += 256) put_q(e / rk, e % rk, qa[((size_t)r * heads + h0) * rk + e]);
+    for (int hh = warp; hh < nh; hh += DTH / 32) {
+        const float4 *src = reinterpret_cast<const float4 *>(qa + ((size_t)r * heads + h0 + hh) * rk);
+#pragma unroll 4
+        for (int i = lane; i < rk / 4; i += 32) {
+            const float4 v = src[i];
+            const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+            const __nv_bfloat162 c = __floats2bfloat162_rn(v.x - __bfloat162float(a.x), v.y - __bfloat162float(a.y)),
+                                 d = __floats2bfloat162_rn(v.z - __bfloat162float(b.x), v.w - __bfloat162float(b.y));
+            *reinterpret_cast<uint2 *>(q_s + hh * ldk + 8 * i) = make_uint2(*reinterpret_cast<const uint32_t *>(&a), *reinterpret_cast<const uint32_t *>(&b));
+            *reinterpret_cast<uint2 *>(q_s + (16 + hh) * ldk + 8 * i) = make_uint2(*reinterpret_cast<const uint32_t *>(&c), *reinterpret_cast<const uint32_t *>(&d));
+        }
+    }
     const int half = rd / 2;
-    for (int e = threadIdx.x; e < nh * half; e += 256) {
+    for (int e = threadIdx.x; e < nh * half; e += DTH) {
         const int hh = e / half, i = e % half;
         const bf16 *src = q + ((size_t)r * heads + h0 + hh) * (dim + rd) + dim;
         const size_t ti = (size_t)min(p, max_seq - 1) * half + i;
@@ -313,7 +341,20 @@ latent_decode_kernel(const float *__restrict__ qa, const bf16 *__restrict__ q, c
     float o[2 * OPW][4];
 #pragma unroll
     for (int i = 0; i < 2 * OPW; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-    const uint32_t a_off = (uint32_t)(((lane & 7) + 8 * ((lane >> 3) & 1)) * ldk + 16 * (lane >> 4));
+    __syncthreads();
+    // this warp's slice of the query
+    uint32_t ah[KPW][4], al[KPW][4];
+    const int ksteps = row16 / 16, kpw = (ksteps + 7) / 8, ks0 = (warp & 7) * kpw, khalf = (warp >> 3) * (DT / 2), nks = max(0, min(kpw, ksteps - ks0));
+#pragma unroll
+    for (int i = 0; i < KPW; ++i) {
+        ah[i][0] = ah[i][1] = ah[i][2] = ah[i][3] = al[i][0] = al[i][1] = al[i][2] = al[i][3] = 0u;
+        if (i < nks) {
+            const uint32_t a = qb + (uint32_t)(((lane & 7) + 8 * ((lane >> 3) & 1)) * ldk + 16 * (lane >> 4) + 32 * (ks0 + i));
+            ldsm4(a, ah[i]);
+            ldsm4(a + 16 * ldk, al[i]);
+        }
+    }
+    __syncthreads();  // the planes make room for the partial scores
     int buf = 0;
     for (int t = rank; t < tiles; t += cl, buf ^= 1) {
         if (t + cl < tiles) {
@@ -323,52 +364,49 @@ latent_decode_kernel(const float *__restrict__ qa, const bf16 *__restrict__ q, c
             asm volatile("cp.async.wait_group 0;" ::: "memory");
         }
         __syncthreads();
-        // ---- scores: eight keys per warp
+        // ---- partial scores of half of the keys
         {
-            float s[4][4];  // hi and lo of even and odd k-steps: four chains of dependent products
+            float s[DT / 16][4];
 #pragma unroll
-            for (int i = 0; i < 4; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
-            // one ldmatrix brings the warp's eight keys for two k-steps
-            const uint32_t bk = kb + (uint32_t)((buf * DT + warp * 8 + (lane & 7)) * ldk + 16 * (lane >> 3));
-#pragma unroll 2
-            for (int ks = 0; ks < row16 / 16; ks += 2) {
-                uint32_t b[4], ah[4], al[4];
-                ldsm4(bk + 32 * ks, b);  // (an odd last k-step reads past its columns; unused)
-                ldsm4(qb + a_off + 32 * ks, ah);
-                ldsm4(qb + 16 * ldk + a_off + 32 * ks, al);
-                mma_bf16(s[0], ah, b[0], b[1]);
-                mma_bf16(s[1], al, b[0], b[1]);
-                if (ks + 1 < row16 / 16) {
-                    ldsm4(qb + a_off + 32 * ks + 32, ah);
-                    ldsm4(qb + 16 * ldk + a_off + 32 * ks + 32, al);
-                    mma_bf16(s[2], ah, b[2], b[3]);
-                    mma_bf16(s[3], al, b[2], b[3]);
+            for (int i = 0; i < DT / 16; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
+            const uint32_t bk = kb + (uint32_t)((buf * DT + khalf + (lane & 7) + 8 * (lane >> 4)) * ldk + 16 * ((lane >> 3) & 1) + 32 * ks0);
+#pragma unroll
+            for (int i = 0; i < KPW; ++i)
+                if (i < nks) {
+#pragma unroll
+                    for (int np = 0; np < DT / 32; ++np) {
+                        uint32_t b[4];
+                        ldsm4(bk + (uint32_t)(np * 16 * ldk + 32 * i), b);
+                        mma_bf16(s[2 * np], al[i], b[0], b[1]), mma_bf16(s[2 * np + 1], al[i], b[2], b[3]);
+                        mma_bf16(s[2 * np], ah[i], b[0], b[1]), mma_bf16(s[2 * np + 1], ah[i], b[2], b[3]);
+                    }
                 }
-            }
+            float *d = sc + ((warp & 7) * 16 + g) * DLS + khalf + 2 * tg;
 #pragma unroll
-            for (int i = 0; i < 4; ++i) s[0][i] = (s[0][i] + s[2][i]) + (s[1][i] + s[3][i]);
-            const int key = warp * 8 + 2 * tg;
-            const bool i0 = t * DT + key < n, i1 = t * DT + key + 1 < n;
-            sc[g * 66 + key] = i0 ? s[0][0] * scale : -INFINITY, sc[g * 66 + key + 1] = i1 ? s[0][1] * scale : -INFINITY;
-            sc[(g + 8) * 66 + key] = i0 ? s[0][2] * scale : -INFINITY, sc[(g + 8) * 66 + key + 1] = i1 ? s[0][3] * scale : -INFINITY;
+            for (int i = 0; i < DT / 16; ++i) {
+                *reinterpret_cast<float2 *>(d + 8 * i) = make_float2(s[i][0], s[i][1]);
+                *reinterpret_cast<float2 *>(d + 8 * DLS + 8 * i) = make_float2(s[i][2], s[i][3]);
+            }
         }
         __syncthreads();
-        // ---- running softmax: two heads per warp
+        // ---- running softmax: a head per warp
+        {
+            float s0 = 0.f, s1 = 0.f;
 #pragma unroll
-        for (int i = 0; i < 2; ++i) {
-            const int hh = warp * 2 + i;
-            const float s0 = sc[hh * 66 + lane], s1 = sc[hh * 66 + lane + 32];
+            for (int w = 0; w < 8; ++w) s0 += sc[(w * 16 + warp) * DLS + lane], s1 += sc[(w * 16 + warp) * DLS + lane + 32];
+            s0 = t * DT + lane < n ? s0 * scale : -INFINITY, s1 = t * DT + lane + 32 < n ? s1 * scale : -INFINITY;
+            const float before = row_m[warp];
             float m = fmaxf(s0, s1);
 #pragma unroll
             for (int d = 16; d > 0; d >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, d));
-            m = fmaxf(m, row_m[hh]);  // every tile holds a key, so the maximum is finite
+            m = fmaxf(m, before);  // every tile holds a key, so the maximum is finite
             const float e0 = expf(s0 - m), e1 = expf(s1 - m);
             const float l = smc_group_sum<32>(e0 + e1);
-            bf16 *pp = reinterpret_cast<bf16 *>(p_s) + hh * 72;
+            bf16 *pp = reinterpret_cast<bf16 *>(p_s) + warp * 72;
             pp[lane] = __float2bfloat16_rn(e0), pp[lane + 32] = __float2bfloat16_rn(e1);
             if (lane == 0) {
-                const float f = expf(row_m[hh] - m);
-                row_f[hh] = f, row_m[hh] = m, row_l[hh] = fmaf(row_l[hh], f, l);
+                const float f = expf(before - m);
+                row_f[warp] = f, row_m[warp] = m, row_l[warp] = fmaf(row_l[warp], f, l);
             }
         }
         __syncthreads();
@@ -381,7 +419,7 @@ latent_decode_kernel(const float *__restrict__ qa, const bf16 *__restrict__ q, c
             ldsm4(pb + (uint32_t)(((lane & 7) + 8 * ((lane >> 3) & 1)) * 144 + 16 * (lane >> 4) + 32 * ks), a);
 #pragma unroll
             for (int i = 0; i < OPW; ++i) {
-                const int grp = warp + 8 * i;
+                const int grp = warp + DTH / 32 * i;
                 if (16 * grp < rk) {
                     uint32_t b[4];
                     ldsm4t(kb + (uint32_t)((buf * DT + ks * 16 + (lane & 7) + 8 * ((lane >> 3) & 1)) * ldk + 32 * grp + 16 * (lane >> 4)), b);
@@ -397,7 +435,7 @@ latent_decode_kernel(const float *__restrict__ qa, const bf16 *__restrict__ q, c
     const int ldp = rk + 4;
 #pragma unroll
     for (int i = 0; i < OPW; ++i) {
-        const int grp = warp + 8 * i;
+        const int grp = warp + DTH / 32 * i;
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
             const int c = 16 * grp + 8 * j + 2 * tg;
@@ -435,7 +473,7 @@ latent_decode_kernel(const float *__restrict__ qa, const bf16 *__restrict__ q, c
     }
     __syncthreads();
     const int per = (rk + cl - 1) / cl, c0 = rank * per, c1 = min(rk, c0 + per);
-    for (int e = threadIdx.x; e < nh * per; e += 256) {
+    for (int e = threadIdx.x; e < nh * per; e += DTH) {
         const int hh = e / per, c = c0 + e % per;
         if (c >= c1) continue;
         float x[DCL], v = 0.f;
@@ -451,8 +489,8 @@ latent_decode_kernel(const float *__restrict__ qa, const bf16 *__restrict__ q, c
 size_t decode_smem(const smc_latent_dims &d)
 {
     const int row16 = (d.kv_rank + d.rot_dim + 15) & ~15, ldk = (row16 + 8) * 2;
-    const size_t tiles = (size_t)(2 * 16 + 2 * DT) * ldk, merged = (size_t)2 * 16 * ldk + (size_t)16 * (d.kv_rank + 4) * 4;
-    return (tiles > merged ? tiles : merged) + 16 * 66 * 4 + 16 * 72 * 2 + 64;
+    const size_t tiles = (size_t)2 * DT * ldk, merged = (size_t)16 * (d.kv_rank + 4) * 4;
+    return decode_head_bytes(ldk) + (tiles > merged ? tiles : merged) + 16 * 72 * 2 + 64;
 }
 
 // ukt[h][c][d] = W_uk[h * dim + d][c]
@@ -490,17 +528,25 @@ __global__ void __launch_bounds__(128) latent_prefill_kernel(const bf16 *__restr
     const int key_lo = (window > 0 ? max(0, p_first - window + 1) : 0) - k0;        // keys as indices from k0
     const int key_hi = p_last - k0;                                                // inclusive; < nk
     const int ldkv = heads * (dim + vdim), ldc = rk + rd;
-    const int cu = dim / 8, cr = rd / 8, cv = vdim / 8, per = cu + cr + cv;
+    const int cu = dim / 8, cr = rd / 8, cv = vdim / 8;
+    // rows of a matrix piece -> tile, 16 bytes per thread and copy; keys past the last visible one become zeros
+    auto copy = [&](uint32_t dst, int ldd, const bf16 *src, int lds, int pieces, int lanes, int start) {
+        const int c0 = threadIdx.x & (lanes - 1), j0 = threadIdx.x / lanes, js = 128 / lanes;
+        for (int c = c0; c < pieces; c += lanes) {
+            const bf16 *p = src + (size_t)(start + j0) * lds + 8 * c;
+            uint32_t d = dst + (uint32_t)(j0 * ldd + 16 * c);
+#pragma unroll 4
+            for (int j = j0; j < KT; j += js, p += (size_t)js * lds, d += (uint32_t)(js * ldd)) {
+                const bool in = start + j <= key_hi;
+                cp16(d, in ? p : src, in);
+            }
+        }
+    };
     auto fetch = [&](int start, int buf) {
         const uint32_t kb = sk + (uint32_t)buf * KT * ldk, vb = sv + (uint32_t)buf * KT * ldv;
-        for (int e = threadIdx.x; e < KT * per; e += 128) {
-            const int j = e / per, c = e % per, key = start + j;
-            const bool in = key <= key_hi;
-            const size_t kk = (size_t)(in ? key : key_hi);
-            if (c < cu) cp16(kb + j * ldk + 16 * c, kv + kk * ldkv + h * dim + 8 * c, in);
-            else if (c < cu + cr) cp16(kb + j * ldk + 16 * c, keys + kk * ldc + rk + 8 * (c - cu), in);
-            else cp16(vb + j * ldv + 16 * (c - cu - cr), kv + kk * ldkv + heads * dim + h * vdim + 8 * (c - cu - cr), in);
-        }
+        copy(kb, ldk, kv + h * dim, ldkv, cu, 16, start);
+        copy(kb + 16 * cu, ldk, keys + rk, ldc, cr, 8, start);
+        copy(vb, ldv, kv + heads * dim + h * vdim, ldkv, cv, 16, start);
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     fetch(key_lo, 0);
@@ -522,12 +568,15 @@ __global__ void __launch_bounds__(128) latent_prefill_kernel(const bf16 *__restr
         dst[half + i] = __float2bfloat16_rn(__fadd_rn(__fmul_rn(v, c), __fmul_rn(u, s)));
     }
 
+    const int tile_hi = p_first - k0, tile_lo = window > 0 ? p_first + QR - window - k0 : -k0;  // keys all of the CTA's queries see
     // rows g and g + 8 of the warp's sixteen; the keys each sees, as indices
     const int r0 = warp * 16 + g, r1 = r0 + 8;
     int hi0 = -1, hi1 = -1, lo0 = 0, lo1 = 0;
     if (t0 + r0 < T) hi0 = p_first + r0 - k0, lo0 = window > 0 ? max(0, p_first + r0 - window + 1) - k0 : -k0;
     if (t0 + r1 < T) hi1 = p_first + r1 - k0, lo1 = window > 0 ? max(0, p_first + r1 - window + 1) - k0 : -k0;
-    const float s0 = sink ? sink[h] : -INFINITY;
+    constexpr float LOG2E = 1.4426950408889634f;
+    const float scale2 = scale * LOG2E;  // scores, maxima and the sink in powers of two
+    const float s0 = sink ? sink[h] * LOG2E : -INFINITY;
     float m0 = s0, m1 = s0, l0 = sink ? 1.f : 0.f, l1 = l0;
     // (with a sink the running pair (maximum, sum) starts as that of the one extra term)
     float o[VT][4];
@@ -563,14 +612,22 @@ __global__ void __launch_bounds__(128) latent_prefill_kernel(const bf16 *__restr
             }
         }
         float tm0 = -INFINITY, tm1 = -INFINITY;
+        if (start >= tile_lo && start + KT - 1 <= tile_hi) {  // every query of the CTA sees the whole tile
 #pragma unroll
-        for (int n = 0; n < KT / 8; ++n) {
+            for (int n = 0; n < KT / 8; ++n) {
+                s[n][0] *= scale2, s[n][1] *= scale2, s[n][2] *= scale2, s[n][3] *= scale2;
+                tm0 = fmaxf(tm0, fmaxf(s[n][0], s[n][1])), tm1 = fmaxf(tm1, fmaxf(s[n][2], s[n][3]));
+            }
+        } else {
 #pragma unroll
-            for (int i = 0; i < 2; ++i) {
-                const int key = start + 8 * n + 2 * tg + i;
-                s[n][i] = key >= lo0 && key <= hi0 ? s[n][i] * scale : -INFINITY;
-                s[n][2 + i] = key >= lo1 && key <= hi1 ? s[n][2 + i] * scale : -INFINITY;
-                tm0 = fmaxf(tm0, s[n][i]), tm1 = fmaxf(tm1, s[n][2 + i]);
+            for (int n = 0; n < KT / 8; ++n) {
+#pragma unroll
+                for (int i = 0; i < 2; ++i) {
+                    const int key = start + 8 * n + 2 * tg + i;
+                    s[n][i] = key >= lo0 && key <= hi0 ? s[n][i] * scale2 : -INFINITY;
+                    s[n][2 + i] = key >= lo1 && key <= hi1 ? s[n][2 + i] * scale2 : -INFINITY;
+                    tm0 = fmaxf(tm0, s[n][i]), tm1 = fmaxf(tm1, s[n][2 + i]);
+                }
             }
         }
         tm0 = fmaxf(tm0, __shfl_xor_sync(0xffffffffu, tm0, 1)), tm0 = fmaxf(tm0, __shfl_xor_sync(0xffffffffu, tm0, 2));
@@ -578,12 +635,12 @@ __global__ void __launch_bounds__(128) latent_prefill_kernel(const bf16 *__restr
         const float nm0 = fmaxf(m0, tm0), nm1 = fmaxf(m1, tm1);
         // a row that has seen nothing yet keeps maximum -inf; its weights are 0
         const float b0 = nm0 > -INFINITY ? nm0 : 0.f, b1 = nm1 > -INFINITY ? nm1 : 0.f;
-        const float c0 = expf(m0 - b0), c1 = expf(m1 - b1);
+        const float c0 = ex2(m0 - b0), c1 = ex2(m1 - b1);
         float ps0 = 0.f, ps1 = 0.f;
         uint32_t p[KT / 16][4];
 #pragma unroll
         for (int n = 0; n < KT / 8; ++n) {
-            const float e0 = expf(s[n][0] - b0), e1 = expf(s[n][1] - b0), e2 = expf(s[n][2] - b1), e3 = expf(s[n][3] - b1);
+            const float e0 = ex2(s[n][0] - b0), e1 = ex2(s[n][1] - b0), e2 = ex2(s[n][2] - b1), e3 = ex2(s[n][3] - b1);
             ps0 += e0 + e1, ps1 += e2 + e3;
             p[n >> 1][(n & 1) * 2] = pack2(e0, e1), p[n >> 1][(n & 1) * 2 + 1] = pack2(e2, e3);
         }
@@ -661,13 +718,13 @@ int attend_absorbed_mma(smc_ctx *ctx, const smc_latent_dims &d, const smc_latent
     while (cl > 1 && ((long long)rw.n * groups * cl > ctx->sm_count || cl / 2 >= most)) cl /= 2;
     auto go = [&](auto kernel) {
         SMC_CUDA(ctx, cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-        smc_launch_dep_cluster(ctx->use_pdl, cl, kernel, dim3(cl, groups, rw.n), dim3(256), smem, s, (const float *)b.qa, (const bf16 *)b.q,
+        smc_launch_dep_cluster(ctx->use_pdl, cl, kernel, dim3(cl, groups, rw.n), dim3(DTH), smem, s, (const float *)b.qa, (const bf16 *)b.q,
                                (const bf16 *)b.cache, (bf16 *)b.oc, rw, sink, cosT, sinT, d.heads, d.dim, d.kv_rank, d.rot_dim, d.ring, d.window, d.scale,
                                max_seq);
         SMC_LAUNCH_CHECK(ctx);
         return (int)SMC_OK;
     };
-    rc = d.kv_rank <= 128 ? go(latent_decode_kernel<1>) : (d.kv_rank <= 256 ? go(latent_decode_kernel<2>) : go(latent_decode_kernel<4>));
+    rc = d.kv_rank <= 256 ? go(latent_decode_kernel<1>) : go(latent_decode_kernel<2>);
     if (rc) return rc;
     o.y = b.o, o.ldy = d.heads * d.vdim, o.y_bf16 = 1;
     const bf16 *wuv = reinterpret_cast<const bf16 *>(w_ukv->d_raw) + (size_t)d.heads * d.dim * d.kv_rank;
@@ -700,7 +757,7 @@ bool smc_latent_prefill_supported(const smc_latent_dims &d)
 
 bool smc_latent_decode_supported(const smc_latent_dims &d)
 {
-    return d.dim % 8 == 0 && d.kv_rank % 8 == 0 && d.rot_dim % 8 == 0 && d.kv_rank <= 512 && decode_smem(d) <= 220 * 1024;
+    return d.dim % 8 == 0 && d.kv_rank % 8 == 0 && d.rot_dim % 8 == 0 && d.kv_rank <= 512 && d.kv_rank + d.rot_dim <= 8 * KPW * 16 && decode_smem(d) <= 220 * 1024;
 }
 
 int smc_latent_transpose_uk(smc_ctx *ctx, const smc_latent_dims &d, const smc_weight *w_ukv, void *out, cudaStream_t s)

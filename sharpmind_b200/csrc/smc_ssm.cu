@@ -87,22 +87,29 @@ __global__ void __launch_bounds__(128) ssm_conv_kernel(const T *__restrict__ zx,
         float hist[TAPS ? TAPS : 1][V];  // hist[j]: input of row r - taps + 1 + j
 #pragma unroll
         for (int j = 0; j < TAPS - 1; ++j) input(r0 - TAPS + 1 + j, hist[j + 1]);
-#pragma unroll 4
-        for (int r = r0; r < r1; ++r) {
+        for (int rb = r0; rb < r1; rb += 8) {
+            typename Pack<T, V>::type raw[8];
 #pragma unroll
-            for (int j = 0; j < TAPS - 1; ++j)
+            for (int k = 0; k < 8; ++k)
+                if (rb + k < r1) raw[k] = *reinterpret_cast<const typename Pack<T, V>::type *>(zx + (size_t)(rb + k) * ld + inner + c);
 #pragma unroll
-                for (int i = 0; i < V; ++i) hist[j][i] = hist[j + 1][i];
-            input(r, hist[TAPS - 1]);
-            float v[V];
+            for (int k = 0; k < 8; ++k) {
+                if (rb + k >= r1) break;
 #pragma unroll
-            for (int i = 0; i < V; ++i) {
-                v[i] = bias[i];
+                for (int j = 0; j < TAPS - 1; ++j)
 #pragma unroll
-                for (int j = 0; j < TAPS; ++j) v[i] = fmaf(wc[i][j], hist[j][i], v[i]);
-                v[i] = silu_for<T>(v[i]);
+                    for (int i = 0; i < V; ++i) hist[j][i] = hist[j + 1][i];
+                float v[V];
+#pragma unroll
+                for (int i = 0; i < V; ++i) {
+                    hist[TAPS - 1][i] = to_f(reinterpret_cast<const T *>(&raw[k])[i]);
+                    v[i] = bias[i];
+#pragma unroll
+                    for (int j = 0; j < TAPS; ++j) v[i] = fmaf(wc[i][j], hist[j][i], v[i]);
+                    v[i] = silu_for<T>(v[i]);
+                }
+                store_v<T, V>(out + (size_t)(rb + k) * ch + c, v);
             }
-            store_v<T, V>(out + (size_t)r * ch + c, v);
         }
     } else {
         for (int r = r0; r < r1; ++r) {
@@ -244,9 +251,9 @@ constexpr int CQ = 64, CP = 32, CTH = 512;
 struct ChunkSmem {  // byte offsets; rows are padded to an odd number of 16-byte units
     int ldn, cb, x, m, xw, st, f, total;
 };
-__host__ __device__ inline ChunkSmem chunk_smem(int N)
+__host__ __device__ constexpr ChunkSmem chunk_smem(int N)
 {
-    ChunkSmem o;
+    ChunkSmem o{};
     const int n16 = (N + 15) & ~15;
     o.ldn = (n16 + 8) * 2;
     o.cb = 0;                                   // two buffers of C [64][N] then B [64][N]
@@ -260,12 +267,13 @@ __host__ __device__ inline ChunkSmem chunk_smem(int N)
 }
 
 // 16 warps: token tile warp % 4 against a quarter of the other side.
-template <int NTW>  // state tiles of 8 columns per warp (eight warps across N)
+template <int NTW, int NC>  // state tiles of 8 columns per warp (eight warps across N); N if known, 0: any up to 64 NTW
 __global__ void __launch_bounds__(CTH) ssm_chunk_kernel(const bf16 *__restrict__ xbc, const float *__restrict__ dt_raw, float *__restrict__ y,
                                                         float *__restrict__ state, smc_rows rw, const float *__restrict__ dt_bias,
-                                                        const float *__restrict__ a_log, const float *__restrict__ d_skip, int heads, int P, int N,
+                                                        const float *__restrict__ a_log, const float *__restrict__ d_skip, int heads, int P, int N_,
                                                         int groups)
 {
+    const int N = NC ? NC : N_;
     extern __shared__ __align__(16) uint8_t csm[];
     const ChunkSmem L = chunk_smem(N);
     const uint32_t sb = (uint32_t)__cvta_generic_to_shared(csm);
@@ -280,9 +288,13 @@ __global__ void __launch_bounds__(CTH) ssm_chunk_kernel(const bf16 *__restrict__
     const float D = d_skip[h], bias = dt_bias[h];
     const double A2 = -(double)expf(a_log[h]) * 1.4426950408889634;  // log decays are kept as powers of two
     const int cn = N / 8, cx = min(CP, P - p0) / 8, per = 2 * cn + cx;
+    const int ft0 = threadIdx.x / per, fc0 = threadIdx.x % per, fts = CTH / per, fcs = CTH % per;  // the copies' (token, piece), stepped without divisions
     auto fetch = [&](int t0, int buf) {
-        for (int e = threadIdx.x; e < CQ * per; e += CTH) {
-            const int t = e / per, c = e % per;
+        for (int t = ft0, c = fc0; t < CQ; t += fts, c += fcs) {
+            if (c >= per) {
+                c -= per;
+                if (++t >= CQ) break;
+            }
             const bool in = t0 + t < T;
             const bf16 *src = xbc + (size_t)(in ? t0 + t : T - 1) * ch;
             if (c < cn) cp16(sb + L.cb + (uint32_t)((2 * buf * CQ + t) * L.ldn + 16 * c), src + inner + (groups + grp) * N + 8 * c, in);
@@ -366,6 +378,7 @@ __global__ void __launch_bounds__(CTH) ssm_chunk_kernel(const bf16 *__restrict__
 #pragma unroll
         for (int i = 0; i < 2; ++i) G[i][0] = G[i][1] = G[i][2] = G[i][3] = Y[i][0] = Y[i][1] = Y[i][2] = Y[i][3] = 0.f;
         const bool any = nq <= mt;  // else every source lies after every token
+#pragma unroll
         for (int k = 0; k < ksteps; k += 2) {
             uint32_t sh[4], sl[4];  // eight state rows for two k-steps (of an odd last pair only the first half is used)
             ldsm4(sb + L.st + (uint32_t)((8 * nq + (lane & 7)) * L.ldn + 32 * k + 16 * (lane >> 3)), sh);
@@ -532,7 +545,9 @@ int recur_chunks(smc_ctx *ctx, const smc_ssm_dims &d, const smc_ssm_bufs &b, con
         SMC_LAUNCH_CHECK(ctx);
         return (int)SMC_OK;
     };
-    return d.state <= 128 ? go(ssm_chunk_kernel<2>) : go(ssm_chunk_kernel<4>);
+    if (d.state == 128) return go(ssm_chunk_kernel<2, 128>);
+    if (d.state == 64) return go(ssm_chunk_kernel<2, 64>);
+    return d.state <= 128 ? go(ssm_chunk_kernel<2, 0>) : go(ssm_chunk_kernel<4, 0>);
 }
 
 template <typename T>
