@@ -469,3 +469,65 @@ def test_folder_command_line_and_trace(cuda, tmp_path):
         for step, places in ((0, [3, 19]), (2, [22, 29])):
             got = np.fromfile(out / f"{step}.f32", "<f4").reshape(2, -1)
             assert rel_err_max(got, logits[places]) < TOL[act]
+
+
+# ---------------------------------------------------------------------------------------- head sizes of real models
+def test_wide_heads_many_tiles(cuda):
+    """Large heads and latents, several key tiles per CTA, two head groups, several chunks of states."""
+    cfg = lu.config([lu.latent(heads=18, dim=128, rot_dim=64, vdim=128, kv_rank=512, q_rank=96, window=333, scale=0.09, rot=lu.yarn(dims=64)),
+                     lu.mamba(heads=4, vdim=64, state=128, groups=2, norm_groups=2), lu.mamba(heads=3, vdim=40, state=64, groups=1, norm_groups=5)],
+                    width=128, vocab=128)
+    t16, w = lu.weights(cfg, 21)
+    tk = toks(700, 128, 5)
+    want = lo.forward(cfg, w, tk)
+    m = build(cuda, cfg, t16, BF16, slots=2, max_seq=720, chunk=320)
+    for cuts in ([], [300, 1, 1, 16, 2, 64, 65], [320, 10, 10, 300]):
+        err = lu.rel_err(run(m, tk, cuts), want)
+        assert err.max() < TOL[BF16], (cuts, int(err.argmax()), float(err.max()))
+    m.close()
+
+
+@pytest.mark.parametrize("slots", [5, 9, 18, 40])
+def test_large_batches_decode_like_one(cuda, slots):
+    """One token for each of many sequences: every cluster size of the attention and every width of the matmuls."""
+    import torch
+
+    from sharpmind_b200.layered import POS_NEXT
+    from sharpmind_b200.session import Session
+
+    cfg = lu.config([lu.latent(heads=20, dim=32, rot_dim=16, vdim=32, kv_rank=64, q_rank=48, window=150, rot=lu.yarn(dims=16)), lu.mamba()], width=64)
+    t16, w = lu.weights(cfg, 22)
+    seqs = [toks(n, cfg["vocab"], n) for n in (4, 210, 77)]
+    want = [lo.forward(cfg, w, q)[-1] for q in seqs]
+    m = build(cuda, cfg, t16, BF16, slots=slots, max_seq=256)
+    s = Session(m)
+    for i in range(slots):
+        s.open(i)
+        s.feed(i, seqs[i % 3][:-1])
+    batch = torch.tensor([int(seqs[i % 3][-1]) for i in range(slots)], dtype=torch.int32, device="cuda")
+    got = m.step(batch, POS_NEXT)[0].cpu().numpy()
+    assert rel_err_max(got, np.stack([want[i % 3] for i in range(slots)])) < TOL[BF16]
+    m.close()
+
+
+@pytest.mark.parametrize("act", [F32, BF16])
+def test_norm_parts_differ_from_groups_and_gate_precedes_norm(cuda, act):
+    """A loud gate in one part must not leak into the others' root mean square."""
+    import torch
+
+    cfg = lu.config([lu.mamba(heads=4, vdim=16, state=16, groups=4, norm_groups=2, ff=0)], alpha=0.3)
+    t16, _ = lu.weights(cfg, 23)
+    big = t16["l0.mix.in"].float()
+    big[:32] *= 30.0  # z of the first two heads: the first part of the norm
+    t16["l0.mix.in"] = big.to(torch.bfloat16)
+    w = {k: v.double().numpy() for k, v in t16.items()}
+    tk = toks(70, cfg["vocab"], 6)
+    want = lo.forward(cfg, w, tk)
+    other = json.loads(json.dumps(cfg))
+    for parts in (1, 4):
+        other["layers"][0]["mixer"]["norm_groups"] = parts
+        assert rel_err_max(lo.forward(other, w, tk), want) > 2 * TOL[act]
+    m = build(cuda, cfg, t16, act)
+    for cuts in ([], [33, 1, 2, 3]):
+        assert rel_err_max(run(m, tk, cuts), want) < TOL[act]
+    m.close()
