@@ -35,7 +35,7 @@ along K and its partial sums are exchanged and added in rank order inside the GE
 `--only layered` times the layered decoder (alternating latent attention and Mamba-2 layers, bfloat16) at the sizes of
 LAYERED_SIZES beside the Llama-shaped decoder (Q8_0) of the same width, depth, feed-forward and vocabulary: a 2048-token
 prompt and decode steps at batch 1 and 32; `:decode` / `:prompt` runs one pass of one size without a graph (the form a
-launch list wants), `:ours` leaves the other model out.
+launch list wants; a decode step follows the prompts of its sequences), `:ours` leaves the other model out.
 `--only ...` runs one kernel or section by itself and prints its own JSON line: the commands behind profiles/.
 """
 from __future__ import annotations
@@ -579,9 +579,9 @@ def layered_section(torch, ctx, dev, size: str, batches, steps: int, n_prompt: i
         return row
     if once == "decode":
         for b in batches:
-            t1 = tok[:b].contiguous()
-            m.step(t1, 0)
-            m.step(t1, layered.POS_NEXT)
+            for i in range(b):
+                m.forward_rows(tok.roll(i), 0, i)
+            m.step(tok[:b].contiguous(), layered.POS_NEXT)
         torch.cuda.synchronize()
         return row
 

@@ -170,7 +170,10 @@ def forward(cfg, weights, tokens, collect=None):
     eps, alpha = cfg["norm"]["eps"], cfg["postln_alpha"]
     x = w["embed"][np.asarray(tokens)]
     for i, layer in enumerate(cfg["layers"]):
-        p = f"l{layer.get('weights_of', i)}."
+        owner = i
+        while cfg["layers"][owner].get("weights_of", owner) != owner:
+            owner = cfg["layers"][owner]["weights_of"]
+        p = f"l{owner}."
         x = norm_about_zero(alpha * x + MIXERS[layer["type"]](x, w, p + "mix.", layer["mixer"], eps), w[p + "norm1"], eps)
         if layer.get("mlp"):
             x = norm_about_zero(alpha * x + gated_ffn(x, w, p + "mlp."), w[p + "norm2"], eps)

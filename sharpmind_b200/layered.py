@@ -58,9 +58,15 @@ def read_config(raw: dict) -> dict:
         mlp = e.get("mlp")
         if mlp and mlp.get("kind", "dense") != "dense":
             raise ops.NotSupportedException(f"layer {i}: feed-forward '{mlp['kind']}'")
-        if not 0 <= src < len(raw["layers"]) or "weights_of" in raw["layers"][src]:
-            raise ops.ArgumentException(f"layer {i}: weights of layer {src}")
-        if src != i and raw["layers"][src]["type"] != kind:
+        for _ in range(len(raw["layers"])):  # a shared layer may name one that shares in turn
+            if not 0 <= src < len(raw["layers"]):
+                raise ops.ArgumentException(f"layer {i}: weights of layer {src}")
+            if raw["layers"][src].get("weights_of", src) == src:
+                break
+            src = raw["layers"][src]["weights_of"]
+        else:
+            raise ops.ArgumentException(f"layer {i}: no layer owns its weights")
+        if raw["layers"][src]["type"] != kind:
             raise ops.ArgumentException(f"layer {i} ({kind}) cannot use the weights of layer {src} ({raw['layers'][src]['type']})")
         layers.append({"type": kind, "weights_of": src, "mixer": dict(e["mixer"]), "ffn": int(mlp["ff"]) if mlp else 0})
     return {"vocab": int(raw["vocab"]), "hidden": int(raw["width"]), "eps": float(raw["norm"]["eps"]), "alpha": float(raw["postln_alpha"]),

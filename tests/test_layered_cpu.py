@@ -16,7 +16,9 @@ def test_config_is_read_and_checked():
     c = layered.read_config(cfg)
     assert c["hidden"] == 96 and c["alpha"] == 2.0 and [x["weights_of"] for x in c["layers"]] == [0, 1, 1] and c["layers"][1]["ffn"] == 0
     assert not any(k.startswith("l2.") for k in layered.tensor_shapes(c))
-    for edit in (lambda d: d["layers"][0].update(type="retention"), lambda d: d["layers"][2].update(weights_of=0), lambda d: d["layers"][2].update(weights_of=7),
+    cfg["layers"].append(lu.share(cfg, 2))  # shares what layer 2 shares
+    assert [x["weights_of"] for x in layered.read_config(cfg)["layers"]] == [0, 1, 1, 1]
+    for edit in (lambda d: d["layers"][1].update(weights_of=2), lambda d: d["layers"][0].update(type="retention"), lambda d: d["layers"][2].update(weights_of=0), lambda d: d["layers"][2].update(weights_of=7),
                  lambda d: d["layers"][0]["mlp"].update(kind="experts")):
         bad = json.loads(json.dumps(cfg))
         edit(bad)
