@@ -1,4 +1,5 @@
-"""Plain, slow statement of the layered decoders (latent attention, Mamba-2, norm after the sum) in numpy float64.
+"""Plain, slow statement of the layered decoders in numpy float64: Fitodra (latent attention, Mamba-2, norm after the sum)
+and Molopel (lightning attention, windowed attention beside retention, layer norm before each part).
 
 One function per mechanism, token loops written out, no cache and no batching: the whole sequence is given and every
 position is computed from it.  Nothing here is shared with the product code.
@@ -161,11 +162,110 @@ def gated_ffn(h, w, p):
     return (silu(h @ w[p + "gate"].T) * (h @ w[p + "up"].T)) @ w[p + "down"].T
 
 
-MIXERS = {"latent_attention": latent_attention, "mamba2": mamba2}
+# ---- layer norm, gated feed-forward with the tanh form of GELU
+def layer_norm(x, w, eps):
+    d = x - np.mean(x, axis=-1, keepdims=True)
+    return d / np.sqrt(np.mean(d * d, axis=-1, keepdims=True) + eps) * w
+
+
+def gelu_tanh(z):
+    z = np.asarray(z, F8)
+    return 0.5 * z * (1.0 + np.tanh(math.sqrt(2.0 / math.pi) * (z + 0.044715 * z ** 3)))
+
+
+def gelu_ffn(h, w, p):
+    return (gelu_tanh(h @ w[p + "gate"].T) * (h @ w[p + "up"].T)) @ w[p + "down"].T
+
+
+# ---- linear attention with one fixed decay per head
+def decayed_sum(q, k, v, decay):
+    """q and k [T, heads, n], v [T, heads, m]: o_t = S_t^T q_t with S_t = decay S_(t-1) + k_t v_t^T, S = 0 before the first."""
+    T, H, n = q.shape
+    out = np.zeros((T, H, v.shape[2]), F8)
+    for h in range(H):
+        S = np.zeros((n, v.shape[2]), F8)
+        for t in range(T):
+            S = decay[h] * S + np.outer(k[t, h], v[t, h])
+            out[t, h] = S.T @ q[t, h]
+    return out
+
+
+def lightning(h, w, p, m, eps):
+    T, H = h.shape[0], m["heads"]
+    q, k = (silu(h @ w[p + n].T).reshape(T, H, m["dim"]) for n in "qk")
+    v = silu(h @ w[p + "v"].T).reshape(T, H, m["vdim"])
+    o = decayed_sum(q, k, v, m["decay"]).reshape(T, -1)
+    return (norm_plain(o, w[p + "norm"], eps) * sigmoid(h @ w[p + "g"].T)) @ w[p + "o"].T
+
+
+def retention(h, w, p, m, eps):
+    T, H, n = h.shape[0], m["heads"], m["dim"]
+    rd, pos = m["rot"]["dims"], np.arange(T)
+    freqs, fac = rotary_frequencies(rd, m["rot"]["base"])
+
+    def turn(x):
+        return np.concatenate([rotate_halves(x[..., :rd], pos, freqs, fac), x[..., rd:]], axis=-1)
+
+    q = turn((h @ w[p + "q"].T).reshape(T, H, n))
+    k = turn((h @ w[p + "k"].T).reshape(T, H, n)) * n ** -0.5
+    v = (h @ w[p + "v"].T).reshape(T, H, m["vdim"])
+    o = unit_rms(decayed_sum(q, k, v, m["decay"]), eps).reshape(T, -1)
+    return (o * silu(h @ w[p + "g"].T)) @ w[p + "o"].T
+
+
+# ---- attention over a window with a learned bias per distance
+def distance_bucket(n, rows, reach):
+    """Half of the table's rows stand for one distance each, the rest for logarithmically growing ranges up to `reach`."""
+    half = rows // 2
+    if n < half:
+        return n
+    return min(rows - 1, half + math.floor(math.log(n / half) / math.log(reach / half) * (rows - half)))
+
+
+def biased_window_attention(h, w, p, m, eps):
+    T, H, G = h.shape[0], m["heads"], m["kv_heads"]
+    q = norm_plain((h @ w[p + "q"].T + w[p + "q.b"]).reshape(T, H, m["dim"]), w[p + "q.norm"], eps)
+    k = norm_plain((h @ w[p + "k"].T + w[p + "k.b"]).reshape(T, G, m["dim"]), w[p + "k.norm"], eps)
+    v = (h @ w[p + "v"].T + w[p + "v.b"]).reshape(T, G, m["vdim"])
+    rel = w[p + "rel"]
+    rows = [distance_bucket(n, rel.shape[0], m["bias_max"]) for n in range(T)]
+    dist = np.maximum(np.arange(T)[:, None] - np.arange(T)[None, :], 0)
+    heads = []
+    for i in range(H):
+        g = i // (H // G)
+        bias = np.array([rel[b, i] for b in rows], F8)[dist]
+        heads.append(attend_window_sink((q[:, i] @ k[:, g].T) * m["scale"] + bias, v[:, g], None, m["mask"]["size"]))
+    return np.concatenate(heads, axis=1) @ w[p + "o"].T
+
+
+def side_by_side(h, w, p, m, eps):
+    return (m["left_scale"] * biased_window_attention(h, w, p + "left.", m["left"], eps)
+            + m["right_scale"] * retention(h, w, p + "right.", m["right"], eps))
+
+
+MIXERS = {"latent_attention": latent_attention, "mamba2": mamba2, "lightning": lightning, "parallel": side_by_side}
 
 
 def forward(cfg, weights, tokens, collect=None):
     """Logits [T, vocab] of one sequence.  `collect`: a list that receives the residual stream after every layer."""
+    return {"Fitodra": forward_norm_after, "Molopel": forward_norm_before}[cfg["architecture"]](cfg, weights, tokens, collect)
+
+
+def forward_norm_before(cfg, w, tokens, collect=None):
+    eps = cfg["norm"]["eps"]
+    x = w["embed"][np.asarray(tokens)] * cfg["embedding"]["scale"]
+    for i, layer in enumerate(cfg["layers"]):
+        p = f"l{i}."
+        x = x + MIXERS[layer["type"]](layer_norm(x, w[p + "norm1"], eps), w, p + "mix.", layer["mixer"], eps)
+        if layer.get("mlp"):
+            x = x + gelu_ffn(layer_norm(x, w[p + "norm2"], eps), w, p + "mlp.")
+        if collect is not None:
+            collect.append(x.copy())
+    cap = cfg["logit_softcap"]
+    return cap * np.tanh(layer_norm(x, w["final.norm"], eps) @ w["embed"].T / cap)
+
+
+def forward_norm_after(cfg, weights, tokens, collect=None):
     w = weights
     eps, alpha = cfg["norm"]["eps"], cfg["postln_alpha"]
     x = w["embed"][np.asarray(tokens)]
