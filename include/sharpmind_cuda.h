@@ -435,19 +435,27 @@ SMC_API int smc_medusa_predict_dev(smc_ctx *ctx, const float *d_hidden, const fl
  * the same entry points as the one above: smc_decode_step, smc_forward_last_logits, smc_forward_logits,
  * smc_forward_rows, smc_model_destroy.
  *
- * Layer:  x <- norm(alpha x + mixer(x));  x <- norm(alpha x + ffn(x)), both norms RMS norms whose weight vector is stored
- * as an offset from one (x / rms * (1 + w)).  x is fp32 throughout.  The logits are norm(x) times the embedding table.
+ * Layer, SMC_NORM_AFTER:   x <- norm(alpha x + mixer(x));  x <- norm(alpha x + ffn(x)), both norms RMS norms whose weight
+ * vector is stored as an offset from one (x / rms * (1 + w)).
+ * Layer, SMC_NORM_BEFORE:  x <- x + mixer(norm(x));  x <- x + ffn(norm(x)), the norms layer norms without a bias,
+ * (x - mean) / sqrt(variance + eps) * w.
+ * x is fp32 throughout and starts as the embedding row times embed_scale.  The logits are norm(x) times the embedding
+ * table, then (softcap > 0) softcap * tanh(logit / softcap).
  * Weights are SMC_BF16 handles, vectors fp32 device pointers; layers may share handles, each has its own cache or state.
  *
  * act_dtype SMC_BF16: activations between the matmuls and the latent cache are bfloat16 (mode SMC_ACT_BF16); SMC_F32:
  * everything is fp32 (mode SMC_ACT_F32).  Norms, rotations, scores, softmax, recurrences and x are fp32 in both.
  *
  * A sequence owns slot `seq` of every layer: a latent layer keeps a ring of the last window - 1 + max_chunk positions
- * (compressed key/value row and rotated key part), a state-space layer its fp32 state and the convolution's last inputs.
+ * (compressed key/value row and rotated key part), a state-space layer its fp32 state and the convolution's last inputs, a
+ * head layer a ring of keys and values and the fp32 states of its linear-attention heads.
  * Position 0 starts a sequence over.  A recurrence has no way back: `pos` must be the number of tokens the slot holds
  * (SMC_E_RANGE otherwise).  smc_decode_step with pos = SMC_POS_NEXT takes each slot's next position from the device,
  * so that a captured CUDA graph of the step can be replayed token after token. */
-enum { SMC_MIX_LATENT = 1, SMC_MIX_MAMBA2 = 2 };
+enum { SMC_MIX_LATENT = 1, SMC_MIX_MAMBA2 = 2, SMC_MIX_HEADS = 3 };
+enum { SMC_NORM_AFTER = 0, SMC_NORM_BEFORE = 1 };
+enum { SMC_FFN_SILU = 0, SMC_FFN_GELU_TANH = 1 };
+enum { SMC_GATE_SILU = 0, SMC_GATE_SIGMOID = 1 };
 #define SMC_POS_NEXT (-1)
 /* Rotation angles p * f_i over pairs (i, i + dims/2), f_i = base^(-2i/dims).  factor > 0: YaRN, frequencies whose
  * wavelength exceeds the `original` context are divided by `factor`, with a ramp between the dimensions that turn `fast`
@@ -456,6 +464,28 @@ typedef struct smc_rotation {
     int dims;
     double base, factor, original, fast, slow;
 } smc_rotation;
+/* Softmax attention heads of a head layer (heads = 0: none).  Query head h reads key/value head h / (heads / kv_heads);
+ * window > 0: position i sees i - window + 1 .. i.  q_norm, k_norm [dim]: RMS norm per head with this weight (null: none).
+ * bias (null: none): scores get bias[bucket(i - j) * heads + h] after the scale, `buckets` rows, bucket(n) = n below
+ * buckets / 2, else min(buckets - 1, b + floor(ln(n / b) / ln(bias_max / b) * (buckets - b))) with b = buckets / 2. */
+typedef struct smc_attn_desc {
+    int heads, kv_heads, dim, vdim, window;
+    float scale, out_scale;
+    const float *q_norm, *k_norm, *bias;
+    int buckets;
+    double bias_max;
+} smc_attn_desc;
+/* Linear attention heads of a head layer (heads = 0: none): S_t = decay_h S_{t-1} + k_scale k_t v_t^T, o_t = S_t^T q_t, S
+ * [dim, vdim] in fp32.  silu: q, k and v pass SiLU after their projection.  rot.dims > 0: the first rot.dims elements of q
+ * and k are rotated.  The heads' outputs are RMS normed in norm_parts equal parts (mix_norm: weight [heads * vdim], null:
+ * none), then multiplied by gate(g).  decay: host pointer, [heads]. */
+typedef struct smc_linear_desc {
+    int heads, dim, vdim, silu, norm_parts, gate;
+    float k_scale, out_scale;
+    smc_rotation rot;
+    const double *decay;
+    const float *mix_norm;
+} smc_linear_desc;
 typedef struct smc_layer_desc {
     int mixer;                /* SMC_MIX_* */
     int heads, vdim;          /* both mixers: heads and value width per head */
@@ -474,7 +504,13 @@ typedef struct smc_layer_desc {
     const smc_weight *w_in;   /* [2 heads vdim + 2 groups state + heads, hidden]: z, x, B, C, dt */
     const float *conv_w, *conv_b, *dt_bias, *a_log, *d_skip, *mix_norm;
     const smc_weight *w_out;  /* [hidden, heads * vdim] */
-    /* feed-forward down(SiLU(gate x) * up x); ffn = 0: none */
+    /* SMC_MIX_HEADS: attention heads and linear-attention heads over one input.  w_in [.., hidden] holds the rows of the
+     * attention heads' q, k, v and the linear heads' q, k, v, g in this order (b_in: a bias per row, may be null), w_out
+     * [hidden, attn.heads * attn.vdim + linear.heads * linear.vdim] reads out_scale times the heads' outputs. */
+    smc_attn_desc attn;
+    smc_linear_desc linear;
+    const float *b_in;
+    /* feed-forward down(act(gate x) * up x), act = ffn_act of the model; ffn = 0: none */
     int ffn;
     const smc_weight *w_gu;   /* [2 ffn, hidden] woven by smc_weight_interleave_rows */
     const smc_weight *w_ffn_down;
@@ -486,6 +522,8 @@ typedef struct smc_layered_desc {
     const smc_layer_desc *layers;
     const smc_weight *embedding; /* [vocab, hidden], also the LM head */
     const float *final_norm;
+    int norm_place, ffn_act;     /* SMC_NORM_*, SMC_FFN_* */
+    float embed_scale, softcap;  /* embed_scale 0 means 1; softcap 0: none */
 } smc_layered_desc;
 SMC_API int smc_model_create_layered(smc_ctx *ctx, const smc_layered_desc *desc, int max_batch, smc_model **out);
 /* Tokens of sequence slot `seq` a layered model holds, -1 when only the device knows (after SMC_POS_NEXT steps).
@@ -501,6 +539,9 @@ SMC_API int smc_rope_tables_yarn(smc_ctx *ctx, const smc_rotation *rot, int maxS
  * receives the rows in bfloat16.  The post-norm form of smc_add_rmsnorm_dev. */
 SMC_API int smc_scaled_add_rmsnorm_dev(smc_ctx *ctx, float *d_x, const float *d_y, const float *d_w, void *d_x16, int rows, int n,
                                        float alpha, float w_offset, float eps, void *stream);
+/* out = (x - mean) / sqrt(variance + eps) * w of every row, fp32 or (out_bf16) bfloat16; beside smc_rmsnorm_dev. */
+SMC_API int smc_layernorm_dev(smc_ctx *ctx, const float *d_x, const float *d_w, void *d_out, int out_bf16, int rows, int n, float eps,
+                              void *stream);
 /* Rows of a SMC_BF16 table as fp32: out[i] = row tokens[i]; beside smc_embed_q8_0_dev. */
 SMC_API int smc_embed_bf16_dev(smc_ctx *ctx, const smc_weight *table, const int *d_tokens, int count, float *d_out, void *stream);
 

@@ -127,6 +127,7 @@ SIGNATURES = {
     "smc_model_dump_layers": (c_int, [c_void_p, c_void_p, c_void_p]),
     "smc_rope_tables_yarn": (c_int, [c_void_p, c_void_p, c_int, c_void_p, c_void_p]),
     "smc_scaled_add_rmsnorm_dev": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_float, c_void_p]),
+    "smc_layernorm_dev": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p]),
     "smc_embed_bf16_dev": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p]),
     "smc_verify_greedy_dev": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p]),
     "smc_medusa_predict_dev": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p]),

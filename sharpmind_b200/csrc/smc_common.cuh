@@ -194,13 +194,18 @@ int smc_launch_rmsnorm_row(smc_ctx *, const float *src, const float *w, float *d
                            cudaStream_t s);
 // ---- dense bfloat16 weights (smc_dense.cu) ----
 // Where a dense matmul puts its product [M, N].  Columns from `split` on (if split > 0) go to y32, fp32, stride ld32.
-// woven: the weight's rows are gate / up pairs (2i, 2i + 1) and y receives SiLU(gate) * up, N / 2 columns.
+// woven: the weight's rows are gate / up pairs (2i, 2i + 1) and y receives act(gate) * up, N / 2 columns; 1: SiLU, 2: the
+// tanh form of GELU.  Otherwise, in this order: bias [N] is added, SiLU applied to columns silu_from .. silu_to - 1, the value
+// v becomes softcap * tanh(v / softcap) (softcap > 0), and (accumulate, fp32 y) the sum joins what y holds.
 struct smc_dense_out {
     void *y;
     int ldy;
     int y_bf16;
     float *y32;
     int ld32, split, woven;
+    const float *bias;
+    int silu_from, silu_to, accumulate;
+    float softcap;
 };
 // x [M, K] with row stride ldx, bfloat16 (x_bf16) or fp32; fp32 rows are multiplied in fp32 on the CUDA cores.
 int smc_launch_dense(smc_ctx *, const void *x, int x_bf16, int ldx, const smc_weight *, int M, const smc_dense_out &, cudaStream_t s);
@@ -220,10 +225,13 @@ struct smc_rows {
 // out = x / rms(x) * (w_offset + w) of chosen rows (row r of the output reads row rows[r], or first + r), fp32 or bfloat16
 int smc_launch_rmsnorm_gather(smc_ctx *, const float *x, const int *rows, int first, int n_rows, const float *w, void *out, int out_bf16, int n,
                               float w_offset, float eps, cudaStream_t s);
-// embedding rows as fp32 x (and bfloat16 x16 when not null), and the step's positions: pos [slots] first positions, then
+// embedding rows times `scale` as fp32 x (and bfloat16 x16 when not null), and the step's positions: pos [slots] first positions, then
 // [slots] lengths; a step starts at pos0, or (pos0 < 0) at each slot's length
 int smc_launch_embed_bf16(smc_ctx *, const smc_weight *table, const int *tokens, int count, float *x, void *x16, int *pos, int slots, int seq0,
-                          int pos0, int max_seq, cudaStream_t s);
+                          int pos0, int max_seq, float scale, cudaStream_t s);
+// the same selection of rows through a layer norm without a bias
+int smc_launch_layernorm(smc_ctx *, const float *x, const int *rows, int first, int n_rows, const float *w, void *out, int out_bf16, int n, float eps,
+                         cudaStream_t s);
 // ---- latent attention (smc_latent.cu) ----
 struct smc_latent_dims {
     int heads, dim, rot_dim, vdim, q_rank, kv_rank, window, ring;
@@ -266,6 +274,51 @@ struct smc_ssm_bufs {
 };
 int smc_ssm_mix(smc_ctx *, const smc_ssm_dims &, const smc_ssm_bufs &, const smc_rows &, int bf16, const float *conv_w, const float *conv_b,
                 const float *dt_bias, const float *a_log, const float *d_skip, const float *norm, cudaStream_t s);
+// ---- attention heads over a window (smc_window.cu) ----
+// q [heads, dim] | k [kv_heads, dim] | v [kv_heads, vdim] of a row start at column `col` of in [rows, ld]
+struct smc_attn_dims {
+    int heads, kv_heads, dim, vdim, window, ring, bias_len;
+    float scale, out_scale, eps;
+};
+struct smc_attn_bufs {
+    const void *in;               // [rows, ld]  T
+    int ld, col;
+    void *q;                      // [rows, heads, dim] normed queries  T
+    void *cache;                  // [slots, ring, kv_heads, dim + vdim] normed keys and values  T: position p in row p % ring
+    void *o;                      // column 0 of the output, row stride ldo  T
+    int ldo;
+    const float *q_norm, *k_norm; // [dim], null: no norm
+    const float *bias;            // [heads, bias_len] by distance, null: none
+};
+int smc_attn_check(smc_ctx *, const smc_attn_dims &);
+int smc_attn_mix(smc_ctx *, const smc_attn_dims &, const smc_attn_bufs &, const smc_rows &, int bf16, int pos0, cudaStream_t s);
+// out[h * len + n] = table[bucket(n) * heads + h]
+int smc_attn_expand_bias(smc_ctx *, const float *table, int heads, int buckets, double bias_max, int len, float *out, cudaStream_t s);
+// ---- linear attention heads with a fixed decay (smc_linear.cu) ----
+// q [heads, dim] | k [heads, dim] | v [heads, vdim] | g [heads, vdim] of a row start at column `col` of in [rows, ld]
+struct smc_linear_dims {
+    int heads, dim, vdim, rot_dims, norm_parts, gate;
+    float k_scale, out_scale, eps;
+};
+struct smc_linear_bufs {
+    const void *in;               // [rows, ld]  T
+    int ld, col;
+    void *qk;                     // [rows, 2 heads dim] rotated queries and keys  T (may be null without a rotation)
+    float *y;                     // [rows, heads, vdim]
+    float *part;                  // [chunks, heads, vdim, dim]: what each chunk adds to the state
+    void *start;                  // [chunks, heads, 2, vdim, dim]: the state before each chunk as bfloat16 hi and lo
+    float *state;                 // [slots, heads, vdim, dim]
+    void *o;                      // column 0 of the output, row stride ldo  T
+    int ldo;
+    const double *log2_decay;     // [heads]
+    const float *decay, *mix_norm;
+    const float *cosT, *sinT;     // [max_seq, rot_dims / 2]
+    int max_seq;
+};
+constexpr int SMC_LINEAR_CHUNK = 128;
+bool smc_linear_chunks_supported(const smc_linear_dims &);  // prompts on the tensor cores (part and start needed)
+int smc_linear_check(smc_ctx *, const smc_linear_dims &);
+int smc_linear_mix(smc_ctx *, const smc_linear_dims &, const smc_linear_bufs &, const smc_rows &, int bf16, cudaStream_t s);
 // ---- layered models (smc_layered.cu) ----
 struct smc_layered;
 void smc_layered_free(smc_layered *);

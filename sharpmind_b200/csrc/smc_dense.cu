@@ -8,31 +8,43 @@
 //   dense_tile_kernel     fp32 (or odd-shaped bfloat16) rows, more: 64 x 64 tiles, fp32 FMAs
 //
 // fp32 rows are multiplied in true fp32 (a bfloat16 weight widens exactly).  Every kernel shares one epilogue: plain
-// fp32 or bfloat16 columns, a second fp32 destination for the trailing columns, or SiLU(gate) * up of woven row pairs.
-#include <cuda_bf16.h>
-
+// fp32 or bfloat16 columns, a second fp32 destination for the trailing columns, or act(gate) * up of woven row pairs; before
+// that a bias, SiLU over a range of columns or a soft cap, and a sum into what the destination holds.
+#include "smc_mma.cuh"
 #include "smc_tc.cuh"
-#include "smc_common.cuh"
 
 namespace {
 
-typedef __nv_bfloat16 bf16;
-
-__device__ __forceinline__ float to_f(float v) { return v; }
-__device__ __forceinline__ float to_f(bf16 v) { return __bfloat162float(v); }
-__device__ __forceinline__ float silu(float g) { return __fdiv_rn(g, 1.0f + expf(-g)); }
-
+// gelu_tanh(z) = z / (1 + e^(-2u)), u = sqrt(2/pi) (z + 0.044715 z^3): 1 + tanh u is 2 / (1 + e^(-2u))
+__device__ __forceinline__ float gelu_arg(float z) { return -1.5957691216057308f * z * fmaf(0.044715f * z, z, 1.0f); }
+template <bool FAST>
+__device__ __forceinline__ float act_pair(int woven, float gate, float up)
+{
+    if (woven == 2) return (FAST ? __fdividef(gate, 1.0f + __expf(gelu_arg(gate))) : __fdiv_rn(gate, 1.0f + expf(gelu_arg(gate)))) * up;
+    return silu(gate) * up;
+}
+// what happens to a sum before it is stored
+__device__ __forceinline__ float finish(const smc_dense_out &o, int n, float v)
+{
+    if (o.bias) v += o.bias[n];
+    if (n >= o.silu_from && n < o.silu_to) v = o.y_bf16 ? silu_for<bf16>(v) : silu(v);
+    if (o.softcap > 0.f) v = o.softcap * tanhf(__fdiv_rn(v, o.softcap));
+    return v;
+}
 __device__ __forceinline__ void put(const smc_dense_out &o, int m, int n, float v)
 {
+    v = finish(o, n, v);
     if (o.split > 0 && n >= o.split) o.y32[(size_t)m * o.ld32 + (n - o.split)] = v;
     else if (o.y_bf16) static_cast<bf16 *>(o.y)[(size_t)m * o.ldy + n] = __float2bfloat16_rn(v);
-    else static_cast<float *>(o.y)[(size_t)m * o.ldy + n] = v;
+    else {
+        float *y = static_cast<float *>(o.y) + (size_t)m * o.ldy + n;
+        *y = o.accumulate ? *y + v : v;
+    }
 }
 __device__ __forceinline__ void put_pair(const smc_dense_out &o, int m, int i, float gate, float up)
 {
-    const float v = silu(gate) * up;
-    if (o.y_bf16) static_cast<bf16 *>(o.y)[(size_t)m * o.ldy + i] = __float2bfloat16_rn(v);
-    else static_cast<float *>(o.y)[(size_t)m * o.ldy + i] = v;
+    if (o.y_bf16) static_cast<bf16 *>(o.y)[(size_t)m * o.ldy + i] = __float2bfloat16_rn(act_pair<true>(o.woven, gate, up));
+    else static_cast<float *>(o.y)[(size_t)m * o.ldy + i] = act_pair<false>(o.woven, gate, up);
 }
 
 // ------------------------------------------------------------------------------ few rows, bfloat16
@@ -254,6 +266,7 @@ __global__ void __launch_bounds__(192, 1) dense_tc_kernel(const __grid_constant_
     smc_tc_fence_after();
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     const uint32_t tmem = *reinterpret_cast<volatile uint32_t *>(smem + OFF_PTR);
+    const bool plain = o.bias == nullptr && o.silu_to <= o.silu_from && !(o.softcap > 0.f);
 
     const int mt = (M + TC_M - 1) / TC_M, nt = (N + BN - 1) / BN, tiles = mt * nt, ksteps = (K + TC_K - 1) / TC_K;
     if (warp == 0) {
@@ -317,7 +330,7 @@ __global__ void __launch_bounds__(192, 1) dense_tc_kernel(const __grid_constant_
                     if (o.woven) {
                         float f[8];
 #pragma unroll
-                        for (int i = 0; i < 8; ++i) f[i] = silu(v[2 * i]) * v[2 * i + 1];
+                        for (int i = 0; i < 8; ++i) f[i] = o.y_bf16 ? act_pair<true>(o.woven, v[2 * i], v[2 * i + 1]) : act_pair<false>(o.woven, v[2 * i], v[2 * i + 1]);
                         const int c2 = nc >> 1;
                         if (o.y_bf16 && nc + 16 <= N && (o.ldy & 7) == 0) {
                             __nv_bfloat162 p[4];
@@ -333,6 +346,10 @@ __global__ void __launch_bounds__(192, 1) dense_tc_kernel(const __grid_constant_
                                 }
                         }
                     } else if (nc + 16 <= N && (o.split == 0 || nc + 16 <= o.split) && (o.ldy & 7) == 0) {
+                        if (!plain) {
+#pragma unroll
+                            for (int i = 0; i < 16; ++i) v[i] = finish(o, nc + i, v[i]);
+                        }
                         if (o.y_bf16) {
                             __nv_bfloat162 p[8];
 #pragma unroll
@@ -342,7 +359,14 @@ __global__ void __launch_bounds__(192, 1) dense_tc_kernel(const __grid_constant_
                         } else {
                             float4 *dst = reinterpret_cast<float4 *>(static_cast<float *>(o.y) + (size_t)m * o.ldy + nc);
 #pragma unroll
-                            for (int i = 0; i < 4; ++i) dst[i] = make_float4(v[4 * i], v[4 * i + 1], v[4 * i + 2], v[4 * i + 3]);
+                            for (int i = 0; i < 4; ++i) {
+                                float4 t = make_float4(v[4 * i], v[4 * i + 1], v[4 * i + 2], v[4 * i + 3]);
+                                if (o.accumulate) {
+                                    const float4 b = dst[i];
+                                    t.x += b.x, t.y += b.y, t.z += b.z, t.w += b.w;
+                                }
+                                dst[i] = t;
+                            }
                         }
                     } else {
 #pragma unroll

@@ -585,12 +585,72 @@ __global__ void __launch_bounds__(256) rmsnorm_gather_kernel(const float *__rest
     }
 }
 
-// Rows of a bfloat16 table, widened; the first CTA of a step also moves the sequences on: pos[slot], the position of the
+// Layer norm without a bias: out[r] = (x - mean) / sqrt(variance + eps) * w of row rows ? rows[r] : first + r, the variance
+// from the deviations themselves.  A CTA per row; NV > 0: the row stays in registers, four elements at a time (up to
+// 1024 NV of them); NV = 0: any length, read again for every pass.
+template <int NV>
+__global__ void __launch_bounds__(256) layernorm_kernel(const float *__restrict__ x, const int *__restrict__ rows, int first,
+                                                        const float *__restrict__ w, void *out, int out_bf16, int n, float eps)
+{
+    __shared__ float red[2][32];
+    float4 g[NV ? NV : 1];
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+        const int i = threadIdx.x + 256 * j;
+        g[j] = 4 * i < n ? __ldg(reinterpret_cast<const float4 *>(w) + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    smc_grid_dep_sync();
+    const float *p = x + (size_t)(rows ? rows[blockIdx.x] : first + (int)blockIdx.x) * n;
+    if (NV) {
+        float4 v[NV ? NV : 1];
+        float sum = 0.f, ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int i = threadIdx.x + 256 * j;
+            v[j] = 4 * i < n ? reinterpret_cast<const float4 *>(p)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+            sum += (v[j].x + v[j].y) + (v[j].z + v[j].w);
+        }
+        const float mean = __fdiv_rn(block_sum(sum, red[0]), (float)n);
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            if (4 * (threadIdx.x + 256 * j) >= n) continue;
+            v[j].x -= mean, v[j].y -= mean, v[j].z -= mean, v[j].w -= mean;
+            ss = fmaf(v[j].x, v[j].x, ss), ss = fmaf(v[j].y, v[j].y, ss), ss = fmaf(v[j].z, v[j].z, ss), ss = fmaf(v[j].w, v[j].w, ss);
+        }
+        const float inv = __fdiv_rn(1.0f, sqrtf(__fdiv_rn(block_sum(ss, red[1]), (float)n) + eps));
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+            const int i = threadIdx.x + 256 * j;
+            if (4 * i >= n) continue;
+            const float4 r = make_float4((v[j].x * inv) * g[j].x, (v[j].y * inv) * g[j].y, (v[j].z * inv) * g[j].z, (v[j].w * inv) * g[j].w);
+            if (out_bf16) {
+                const __nv_bfloat162 lo = __floats2bfloat162_rn(r.x, r.y), hi = __floats2bfloat162_rn(r.z, r.w);
+                reinterpret_cast<uint2 *>(static_cast<__nv_bfloat16 *>(out) + (size_t)blockIdx.x * n)[i] =
+                    make_uint2(*reinterpret_cast<const uint32_t *>(&lo), *reinterpret_cast<const uint32_t *>(&hi));
+            } else {
+                reinterpret_cast<float4 *>(static_cast<float *>(out) + (size_t)blockIdx.x * n)[i] = r;
+            }
+        }
+        return;
+    }
+    float sum = 0.f, ss = 0.f;
+    for (int i = threadIdx.x; i < n; i += 256) sum += p[i];
+    const float mean = __fdiv_rn(block_sum(sum, red[0]), (float)n);
+    for (int i = threadIdx.x; i < n; i += 256) ss = fmaf(p[i] - mean, p[i] - mean, ss);
+    const float inv = __fdiv_rn(1.0f, sqrtf(__fdiv_rn(block_sum(ss, red[1]), (float)n) + eps));
+    for (int i = threadIdx.x; i < n; i += 256) {
+        const float v = ((p[i] - mean) * inv) * w[i];
+        if (out_bf16) static_cast<__nv_bfloat16 *>(out)[(size_t)blockIdx.x * n + i] = __float2bfloat16_rn(v);
+        else static_cast<float *>(out)[(size_t)blockIdx.x * n + i] = v;
+    }
+}
+
+// Rows of a bfloat16 table, widened and scaled; the first CTA of a step also moves the sequences on: pos[slot], the position of the
 // step's first row, becomes pos0, or (pos0 < 0) the slot's length, and the length pos[slots + slot] becomes what the
 // slot holds after the step.  A position past the tables raises the status word.
 __global__ void __launch_bounds__(256) embed_bf16_kernel(const __nv_bfloat16 *__restrict__ table, const int *__restrict__ tokens, int H, int vocab,
                                                          float *__restrict__ out, __nv_bfloat16 *__restrict__ out16, int *pos, int slots, int seq0, int pos0,
-                                                         int max_seq, int *status)
+                                                         int max_seq, float scale, int *status)
 {
     smc_grid_dep_sync();
     const int r = blockIdx.x;
@@ -604,9 +664,9 @@ __global__ void __launch_bounds__(256) embed_bf16_kernel(const __nv_bfloat16 *__
     int tok = tokens[r];
     tok = tok < 0 ? 0 : (tok >= vocab ? vocab - 1 : tok);
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
-        const __nv_bfloat16 v = table[(size_t)tok * H + i];
-        out[(size_t)r * H + i] = __bfloat162float(v);
-        if (out16) out16[(size_t)r * H + i] = v;
+        const float v = __bfloat162float(table[(size_t)tok * H + i]) * scale;
+        out[(size_t)r * H + i] = v;
+        if (out16) out16[(size_t)r * H + i] = __float2bfloat16_rn(v);
     }
 }
 
@@ -865,7 +925,13 @@ int smc_embed_bf16_dev(smc_ctx *ctx, const smc_weight *table, const int *d_token
     if (!ctx || !table || !d_tokens || !d_out || count < 0) return smc_fail(ctx, SMC_E_INVALID, "embed: bad arguments");
     if (table->dtype != SMC_BF16) return smc_fail(ctx, SMC_E_UNSUPPORTED, "embed: the table is not bfloat16");
     if (count == 0) return SMC_OK;
-    return smc_launch_embed_bf16(ctx, table, d_tokens, count, d_out, nullptr, nullptr, 0, 0, 0, 1, static_cast<cudaStream_t>(stream));
+    return smc_launch_embed_bf16(ctx, table, d_tokens, count, d_out, nullptr, nullptr, 0, 0, 0, 1, 1.0f, static_cast<cudaStream_t>(stream));
+}
+
+int smc_layernorm_dev(smc_ctx *ctx, const float *d_x, const float *d_w, void *d_out, int out_bf16, int rows, int n, float eps, void *stream)
+{
+    if (!ctx || !d_x || !d_w || !d_out || rows < 0 || n <= 0) return smc_fail(ctx, SMC_E_INVALID, "layernorm: bad arguments");
+    return smc_launch_layernorm(ctx, d_x, nullptr, 0, rows, d_w, d_out, out_bf16, n, eps, static_cast<cudaStream_t>(stream));
 }
 
 }  // extern "C"
@@ -887,11 +953,26 @@ int smc_launch_rmsnorm_gather(smc_ctx *ctx, const float *x, const int *rows, int
     return SMC_OK;
 }
 
+int smc_launch_layernorm(smc_ctx *ctx, const float *x, const int *rows, int first, int n_rows, const float *w, void *out, int out_bf16, int n, float eps,
+                         cudaStream_t s)
+{
+    if (n_rows == 0) return SMC_OK;
+    auto go = [&](auto kernel) { smc_launch_dep(ctx->use_pdl, kernel, dim3(n_rows), dim3(256), 0, s, x, rows, first, w, out, out_bf16, n, eps); };
+    const bool vec = n % 4 == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+    if (vec && n <= 1024) go(layernorm_kernel<1>);
+    else if (vec && n <= 2048) go(layernorm_kernel<2>);
+    else if (vec && n <= 4096) go(layernorm_kernel<4>);
+    else if (vec && n <= 8192) go(layernorm_kernel<8>);
+    else go(layernorm_kernel<0>);
+    SMC_LAUNCH_CHECK(ctx);
+    return SMC_OK;
+}
+
 int smc_launch_embed_bf16(smc_ctx *ctx, const smc_weight *table, const int *tokens, int count, float *x, void *x16, int *pos, int slots, int seq0,
-                          int pos0, int max_seq, cudaStream_t s)
+                          int pos0, int max_seq, float scale, cudaStream_t s)
 {
     smc_launch_dep(ctx->use_pdl, embed_bf16_kernel, dim3(count), dim3(256), 0, s, reinterpret_cast<const __nv_bfloat16 *>(table->d_raw), tokens, table->K,
-                   table->N, x, static_cast<__nv_bfloat16 *>(x16), pos, slots, seq0, pos0, max_seq, ctx->d_status);
+                   table->N, x, static_cast<__nv_bfloat16 *>(x16), pos, slots, seq0, pos0, max_seq, scale, ctx->d_status);
     SMC_LAUNCH_CHECK(ctx);
     return SMC_OK;
 }

@@ -10,28 +10,14 @@
 //              (latent_prefill_kernel): a third of the arithmetic at prompt sizes.
 // The cache is a ring: position p lives in row p % ring, ring >= window - 1 + the longest portion, so the rows a portion
 // writes never displace one that its first query still sees.
-#include <cuda_bf16.h>
 #include <math.h>
 
 #include <type_traits>
 #include <vector>
 
-#include "smc_common.cuh"
+#include "smc_mma.cuh"
 
 namespace {
-
-typedef __nv_bfloat16 bf16;
-
-__device__ __forceinline__ float to_f(float v) { return v; }
-__device__ __forceinline__ float to_f(bf16 v) { return __bfloat162float(v); }
-template <typename T> __device__ __forceinline__ T from_f(float v);
-template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
-template <> __device__ __forceinline__ bf16 from_f<bf16>(float v) { return __float2bfloat16_rn(v); }
-__device__ __forceinline__ void row_place(const smc_rows &rw, int r, int &slot, int &p)
-{
-    slot = rw.seq0 >= 0 ? rw.seq0 : r;
-    p = rw.pos[slot] + (rw.seq0 >= 0 ? r : 0);
-}
 
 // ------------------------------------------------------------------------------ after the down projections
 // A warp per (row, part): the query latent normed, or the key/value latent normed and the shared key part rotated, both
@@ -221,38 +207,6 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const uint4 *__restr
     if (e >= (long long)n * row16) return;
     const int j = (int)(e / row16), c = (int)(e % row16);
     keys[e] = cache[((size_t)slot * ring + (k0 + j) % ring) * row16 + c];
-}
-
-__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1)
-{
-    asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-        : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-        : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void ldsm4(uint32_t addr, uint32_t (&r)[4])
-{
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm4t(uint32_t addr, uint32_t (&r)[4])
-{
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-// 16 bytes global -> shared, zeros when `in` is false (the address must be valid either way)
-__device__ __forceinline__ void cp16(uint32_t dst, const void *src, bool in)
-{
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(in ? 16 : 0) : "memory");
-}
-// 2^x for x <= 0
-__device__ __forceinline__ float ex2(float x)
-{
-    float v;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(v) : "f"(x));
-    return v;
-}
-__device__ __forceinline__ uint32_t pack2(float a, float b)
-{
-    const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
-    return *reinterpret_cast<const uint32_t *>(&v);
 }
 
 // ------------------------------------------------------------------------------ absorbed form on the tensor cores (bfloat16)

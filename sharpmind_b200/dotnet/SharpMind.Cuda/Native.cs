@@ -165,6 +165,8 @@ internal static unsafe partial class Native
     [LibraryImport(Lib)] internal static partial int smc_rope_tables_yarn(nint ctx, nint rotation, int maxSeq, nint dCos, nint dSin);
     [LibraryImport(Lib)] internal static partial int smc_scaled_add_rmsnorm_dev(nint ctx, nint dX, nint dY, nint dW, nint dX16, int rows, int n,
         float alpha, float wOffset, float eps, nint stream);
+    [LibraryImport(Lib)] internal static partial int smc_layernorm_dev(nint ctx, nint dX, nint dW, nint dOut, int outBf16, int rows, int n, float eps,
+        nint stream);
     [LibraryImport(Lib)] internal static partial int smc_embed_bf16_dev(nint ctx, nint table, nint dTokens, int count, nint dOut, nint stream);
 
     // ---- GGUF

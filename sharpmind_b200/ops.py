@@ -557,6 +557,14 @@ class DeviceOps:
                                                    self._chk(out), self._stream()))
         return out
 
+    def layernorm(self, x, w, eps: float, bf16: bool = False):
+        """(x - mean) / sqrt(variance + eps) * w of every row, fp32 or bfloat16."""
+        t, (rows, n) = self.torch, x.shape
+        out = t.empty((rows, n), dtype=t.bfloat16 if bf16 else t.float32, device=x.device)
+        self.ctx.check(self.ctx.lib.smc_layernorm_dev(self.ctx.h, self._chk(x, t.float32), self._chk(w, t.float32), out.data_ptr(), int(bf16), rows, n,
+                                                      C.c_float(eps), self._stream()))
+        return out
+
     def scaled_add_rmsnorm_(self, x, y, w, alpha: float, eps: float, w_offset: float = 1.0, x16=None):
         """x = norm(alpha * x + y) * (w_offset + w) in place (y may be None); `x16` also receives the rows in bfloat16."""
         rows, n = x.shape

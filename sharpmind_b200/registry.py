@@ -22,6 +22,7 @@ def _layered(ctx, folder, raw, max_seq, max_batch, act, max_chunk):
 # architecture name of config.json -> loader(ctx, folder, config, max_seq, max_batch, act, max_chunk)
 ARCHITECTURES = {
     "Fitodra": _layered,
+    "Molopel": _layered,
 }
 
 
@@ -49,20 +50,25 @@ def describe(path: str) -> str:
     if not os.path.isdir(path):
         return f"{path}: GGUF file"
     from .layered import read_config, tensor_shapes
+    from .safetensors import SafetensorsFile
 
     with open(os.path.join(path, "config.json")) as f:
         raw = json.load(f)
     if raw.get("architecture") not in ARCHITECTURES:
         raise ops.NotSupportedException(f"architecture '{raw.get('architecture')}'")
     cfg = read_config(raw)
+    weights = os.path.join(path, "model.safetensors")
+    held = SafetensorsFile(weights).tensors if os.path.exists(weights) else {}
     params = 0
-    for shape in tensor_shapes(cfg).values():
+    for name, shape in tensor_shapes(cfg).items():
         n = 1
-        for d in shape:
-            n *= d
+        for i, d in enumerate(shape):  # a size the configuration leaves open is the file's
+            n *= d if d is not None else (held[name]["shape"][i] if name in held else 0)
         params += n
     lines = [f"{raw['architecture']}: {len(cfg['layers'])} layers, width {cfg['hidden']}, vocabulary {cfg['vocab']}, {params} parameters"]
     for i, L in enumerate(cfg["layers"]):
         shared = f" (weights of layer {L['weights_of']})" if L["weights_of"] != i else ""
-        lines.append(f"  {i}: {L['type']}, {L['mixer']['heads']} heads, ffn {L['ffn']}{shared}")
+        m = L["mixer"]
+        heads = " + ".join(str(m[k]["heads"]) for k in ("left", "right")) if L["type"] == "parallel" else m["heads"]
+        lines.append(f"  {i}: {L['type']}, {heads} heads, ffn {L['ffn']}{shared}")
     return "\n".join(lines)
