@@ -3,7 +3,7 @@
     python bench.py [--gpus N] [--steps K] [--warmup W] [--impl ours|reference]
                     [--workload llama70b|llama8b] [--batch M] [--mode q8|f32] [--layers L]
                     [--only gemv:<shape>[:<M>[:q8|q8pre|f32[:ring]]] | decode[:qwen3|llama8b][:q8kv] | prompt[:llama8b] | elementwise | prefill
-                            | layered[:<size>][:prompt|decode|ours]]
+                            | layered[:molopel][:<size>][:prompt|decode|ours]]
 
 Workload (default `llama70b`, BASELINE configs[4], the largest configuration that fits one GPU and the one the
 multi-GPU target is stated on): the Llama-3-70B-shaped FFN GEMV stack -- per layer the fused gate||up projection
@@ -35,7 +35,9 @@ along K and its partial sums are exchanged and added in rank order inside the GE
 `--only layered` times the layered decoder (alternating latent attention and Mamba-2 layers, bfloat16) at the sizes of
 LAYERED_SIZES beside the Llama-shaped decoder (Q8_0) of the same width, depth, feed-forward and vocabulary: a 2048-token
 prompt and decode steps at batch 1 and 32; `:decode` / `:prompt` runs one pass of one size without a graph (the form a
-launch list wants; a decode step follows the prompts of its sequences), `:ours` leaves the other model out.
+launch list wants; a decode step follows the prompts of its sequences), `:ours` leaves the other models out.
+`--only layered:molopel` does the same for the other layered design (lightning attention and windowed attention beside
+retention, in turn) beside the first one and the Llama-shaped decoder of equal size.
 `--only ...` runs one kernel or section by itself and prints its own JSON line: the commands behind profiles/.
 """
 from __future__ import annotations
@@ -530,13 +532,34 @@ def layered_config(size: str) -> dict:
     return {"vocab": V, "hidden": H, "eps": 1e-5, "alpha": (2 * L) ** 0.25, "layers": layers}
 
 
+def molopel_config(size: str) -> dict:
+    """The same width, depth, feed-forward, vocabulary and window: lightning attention and windowed attention beside retention
+    in turn, head size 128, four query heads per key/value head, half as many retention heads."""
+    H, L, F, V, heads, _, _, window, _ = LAYERED_SIZES[size]
+
+    def decays(n):
+        return [1.0 - 2.0 ** (-3.0 - 6.0 * i / n) for i in range(n)]
+
+    lit = {"heads": heads, "dim": 128, "vdim": 128, "decay": decays(heads)}
+    par = {"left": {"heads": heads, "kv_heads": heads // 4, "dim": 128, "vdim": 128, "mask": {"size": window}, "scale": 128 ** -0.5, "bias_max": window},
+           "right": {"heads": heads // 2, "dim": 128, "vdim": 128, "rot": {"base": 10000.0, "dims": 128}, "decay": decays(heads // 2)},
+           "left_scale": 0.7, "right_scale": 0.7}
+    layers = [{"type": ("lightning", "parallel")[i & 1], "mixer": (lit, par)[i & 1], "mlp": {"kind": "dense", "ff": F}} for i in range(L)]
+    from sharpmind_b200 import layered
+
+    return layered.read_config({"architecture": "Molopel", "vocab": V, "width": H, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+                                "logit_softcap": 30.0, "layers": layers})
+
+
 class LayeredDeviceWeights:
     """Random bfloat16 tensors of a configuration, drawn on the device when asked for."""
 
     def __init__(self, torch, cfg: dict):
         from sharpmind_b200 import layered
 
-        self.torch, self.shapes = torch, layered.tensor_shapes(cfg)
+        self.torch = torch
+        self.shapes = {k: tuple(32 if n is None else n for n in v) for k, v in layered.tensor_shapes(cfg).items()}
+        self.before = cfg.get("norm_place") == layered.NORM_BEFORE
         self.g = torch.Generator(device="cuda").manual_seed(4321)
 
     def __getitem__(self, name: str):
@@ -546,20 +569,21 @@ class LayeredDeviceWeights:
             x = x * 0.5
         elif last == "mix.dt_bias":
             x = x * 0.5 - 2.0
-        elif last in ("mix.dq.norm", "mix.dkv.norm", "mix.norm"):
+        elif last in ("mix.dq.norm", "mix.dkv.norm", "mix.norm", "mix.left.q.norm", "mix.left.k.norm"):
             x = 1.0 + 0.1 * x
         elif len(shape) == 1:
-            x = 0.1 * x
+            x = (1.0 if self.before and last.startswith("norm") else 0.0) + 0.1 * x
         elif last != "mix.conv":
             x = x * shape[1] ** -0.5
         return x.to(t.bfloat16)
 
 
-def layered_section(torch, ctx, dev, size: str, batches, steps: int, n_prompt: int, once: str = "", ours_only: bool = False) -> dict:
-    """Prompt and decode throughput of the layered decoder, and of the Llama-shaped Q8_0 decoder of equal size."""
+def layered_section(torch, ctx, dev, size: str, batches, steps: int, n_prompt: int, once: str = "", ours_only: bool = False,
+                    molopel: bool = False) -> dict:
+    """Prompt and decode throughput of a layered decoder, and of the Llama-shaped Q8_0 decoder of equal size."""
     from sharpmind_b200 import layered, ops
 
-    cfg = layered_config(size)
+    cfg = molopel_config(size) if molopel else layered_config(size)
     H, L, F, V, heads = LAYERED_SIZES[size][:5]
     weights = LayeredDeviceWeights(torch, cfg)
     max_seq = n_prompt + 4 * steps + 64
@@ -567,7 +591,7 @@ def layered_section(torch, ctx, dev, size: str, batches, steps: int, n_prompt: i
     params = sum(int(np.prod(sh)) for sh in weights.shapes.values())
     g = torch.Generator(device="cuda").manual_seed(7)
     tok = torch.randint(0, V, (n_prompt,), generator=g, device="cuda", dtype=torch.int32)
-    row = {"size": size, "hidden": H, "layers": L, "ffn": F, "vocab": V, "parameters_M": round(params / 1e6, 1)}
+    row = {"size": size, "design": "Molopel" if molopel else "Fitodra", "hidden": H, "layers": L, "ffn": F, "vocab": V, "parameters_M": round(params / 1e6, 1)}
 
     def rewind(b):
         for i in range(b):
@@ -611,6 +635,10 @@ def layered_section(torch, ctx, dev, size: str, batches, steps: int, n_prompt: i
         rewind(b)
     row["device_status"] = ctx.device_status()
     m.close()
+    del weights, m
+    if not ours_only and molopel:
+        other = layered_section(torch, ctx, dev, size, batches, steps, n_prompt, ours_only=True)
+        row["fitodra"] = {k: other[k] for k in ("parameters_M", "prompt", "decode")}
     if not ours_only:
         # Llama-shaped, every matrix Q8_0, head size 128, grouped KV heads
         like = dict(n_layers=L, hidden=H, n_heads=H // 128, n_kv_heads=max(1, H // 256), head_dim=128, ffn=F, vocab=V, max_seq=n_prompt + 64, dtype=8,
@@ -659,7 +687,7 @@ def run_only(args):
         sizes = [p for p in parts[1:] if p in LAYERED_SIZES] or list(LAYERED_SIZES)
         once = next((p for p in parts[1:] if p in ("prompt", "decode")), "")
         batches = [args.batch] if once else [1, 32]
-        res = {"layered": [layered_section(torch, ctx, dev, sz, batches, max(args.steps, 4), 2048, once, "ours" in parts) for sz in sizes]}
+        res = {"layered": [layered_section(torch, ctx, dev, sz, batches, max(args.steps, 4), 2048, once, "ours" in parts, "molopel" in parts) for sz in sizes]}
     else:
         raise SystemExit(f"unknown --only section '{args.only}'")
     print(json.dumps(res), flush=True)

@@ -10,6 +10,8 @@
 // fp32 rows are multiplied in true fp32 (a bfloat16 weight widens exactly).  Every kernel shares one epilogue: plain
 // fp32 or bfloat16 columns, a second fp32 destination for the trailing columns, or act(gate) * up of woven row pairs; before
 // that a bias, SiLU over a range of columns or a soft cap, and a sum into what the destination holds.
+#include <type_traits>
+
 #include "smc_mma.cuh"
 #include "smc_tc.cuh"
 
@@ -17,11 +19,15 @@ namespace {
 
 // gelu_tanh(z) = z / (1 + e^(-2u)), u = sqrt(2/pi) (z + 0.044715 z^3): 1 + tanh u is 2 / (1 + e^(-2u))
 __device__ __forceinline__ float gelu_arg(float z) { return -1.5957691216057308f * z * fmaf(0.044715f * z, z, 1.0f); }
-template <bool FAST>
 __device__ __forceinline__ float act_pair(int woven, float gate, float up)
 {
-    if (woven == 2) return (FAST ? __fdividef(gate, 1.0f + __expf(gelu_arg(gate))) : __fdiv_rn(gate, 1.0f + expf(gelu_arg(gate)))) * up;
-    return silu(gate) * up;
+    return (woven == 2 ? __fdiv_rn(gate, 1.0f + expf(gelu_arg(gate))) : silu(gate)) * up;
+}
+// in front of a bfloat16 rounding
+template <bool GELU>
+__device__ __forceinline__ float act_pair_fast(float gate, float up)
+{
+    return __fdividef(gate, 1.0f + __expf(GELU ? gelu_arg(gate) : -gate)) * up;
 }
 // what happens to a sum before it is stored
 __device__ __forceinline__ float finish(const smc_dense_out &o, int n, float v)
@@ -43,8 +49,9 @@ __device__ __forceinline__ void put(const smc_dense_out &o, int m, int n, float 
 }
 __device__ __forceinline__ void put_pair(const smc_dense_out &o, int m, int i, float gate, float up)
 {
-    if (o.y_bf16) static_cast<bf16 *>(o.y)[(size_t)m * o.ldy + i] = __float2bfloat16_rn(act_pair<true>(o.woven, gate, up));
-    else static_cast<float *>(o.y)[(size_t)m * o.ldy + i] = act_pair<false>(o.woven, gate, up);
+    const float v = act_pair(o.woven, gate, up);
+    if (o.y_bf16) static_cast<bf16 *>(o.y)[(size_t)m * o.ldy + i] = __float2bfloat16_rn(v);
+    else static_cast<float *>(o.y)[(size_t)m * o.ldy + i] = v;
 }
 
 // ------------------------------------------------------------------------------ few rows, bfloat16
@@ -231,8 +238,16 @@ struct TcShape {
     static constexpr uint32_t COLS = 2 * BN;                                       // two accumulators
 };
 
+// What the epilogue does: store (or sum), SiLU or GELU of woven pairs, or everything `finish` knows.
+enum { EPI_STORE, EPI_SILU_PAIRS, EPI_GELU_PAIRS, EPI_FINISH };
+// y[0..3] += v without waiting for y: every element has one writer per launch, so the result does not depend on an order
+__device__ __forceinline__ void add4(float *y, float a, float b, float c, float d)
+{
+    asm volatile("red.global.add.v4.f32 [%0], {%1, %2, %3, %4};" ::"l"(y), "f"(a), "f"(b), "f"(c), "f"(d) : "memory");
+}
+
 // Warp 0: TMA loads; warp 1: MMA issue; warps 2 .. 5: epilogue (one TMEM lane = one token per thread).
-template <int BN>
+template <int BN, int EPI>
 __global__ void __launch_bounds__(192, 1) dense_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w, int M,
                                                           int N, int K, smc_dense_out o, int *status)
 {
@@ -266,7 +281,6 @@ __global__ void __launch_bounds__(192, 1) dense_tc_kernel(const __grid_constant_
     smc_tc_fence_after();
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     const uint32_t tmem = *reinterpret_cast<volatile uint32_t *>(smem + OFF_PTR);
-    const bool plain = o.bias == nullptr && o.silu_to <= o.silu_from && !(o.softcap > 0.f);
 
     const int mt = (M + TC_M - 1) / TC_M, nt = (N + BN - 1) / BN, tiles = mt * nt, ksteps = (K + TC_K - 1) / TC_K;
     if (warp == 0) {
@@ -327,10 +341,16 @@ __global__ void __launch_bounds__(192, 1) dense_tc_kernel(const __grid_constant_
                     float v[16];
 #pragma unroll
                     for (int i = 0; i < 16; ++i) v[i] = __uint_as_float(r[h][i]);
-                    if (o.woven) {
+                    constexpr bool PAIRS = EPI == EPI_SILU_PAIRS || EPI == EPI_GELU_PAIRS;
+                    if (PAIRS) {
                         float f[8];
+                        if (o.y_bf16) {
 #pragma unroll
-                        for (int i = 0; i < 8; ++i) f[i] = o.y_bf16 ? act_pair<true>(o.woven, v[2 * i], v[2 * i + 1]) : act_pair<false>(o.woven, v[2 * i], v[2 * i + 1]);
+                            for (int i = 0; i < 8; ++i) f[i] = act_pair_fast<EPI == EPI_GELU_PAIRS>(v[2 * i], v[2 * i + 1]);
+                        } else {
+#pragma unroll
+                            for (int i = 0; i < 8; ++i) f[i] = act_pair(EPI == EPI_GELU_PAIRS ? 2 : 1, v[2 * i], v[2 * i + 1]);
+                        }
                         const int c2 = nc >> 1;
                         if (o.y_bf16 && nc + 16 <= N && (o.ldy & 7) == 0) {
                             __nv_bfloat162 p[4];
@@ -346,9 +366,25 @@ __global__ void __launch_bounds__(192, 1) dense_tc_kernel(const __grid_constant_
                                 }
                         }
                     } else if (nc + 16 <= N && (o.split == 0 || nc + 16 <= o.split) && (o.ldy & 7) == 0) {
-                        if (!plain) {
+                        if (EPI == EPI_FINISH) {
+                            if (o.bias) {
 #pragma unroll
-                            for (int i = 0; i < 16; ++i) v[i] = finish(o, nc + i, v[i]);
+                                for (int i = 0; i < 4; ++i) {
+                                    const float4 b = __ldg(reinterpret_cast<const float4 *>(o.bias + nc) + i);
+                                    v[4 * i] += b.x, v[4 * i + 1] += b.y, v[4 * i + 2] += b.z, v[4 * i + 3] += b.w;
+                                }
+                            }
+                            if (nc >= o.silu_from && nc + 16 <= o.silu_to && o.y_bf16) {
+#pragma unroll
+                                for (int i = 0; i < 16; ++i) v[i] = silu_for<bf16>(v[i]);
+                            } else if (nc < o.silu_to && nc + 16 > o.silu_from) {
+#pragma unroll
+                                for (int i = 0; i < 16; ++i) v[i] = nc + i >= o.silu_from && nc + i < o.silu_to ? silu(v[i]) : v[i];
+                            }
+                            if (o.softcap > 0.f) {
+#pragma unroll
+                                for (int i = 0; i < 16; ++i) v[i] = o.softcap * tanhf(__fdiv_rn(v[i], o.softcap));
+                            }
                         }
                         if (o.y_bf16) {
                             __nv_bfloat162 p[8];
@@ -360,12 +396,8 @@ __global__ void __launch_bounds__(192, 1) dense_tc_kernel(const __grid_constant_
                             float4 *dst = reinterpret_cast<float4 *>(static_cast<float *>(o.y) + (size_t)m * o.ldy + nc);
 #pragma unroll
                             for (int i = 0; i < 4; ++i) {
-                                float4 t = make_float4(v[4 * i], v[4 * i + 1], v[4 * i + 2], v[4 * i + 3]);
-                                if (o.accumulate) {
-                                    const float4 b = dst[i];
-                                    t.x += b.x, t.y += b.y, t.z += b.z, t.w += b.w;
-                                }
-                                dst[i] = t;
+                                if (o.accumulate) add4(reinterpret_cast<float *>(dst + i), v[4 * i], v[4 * i + 1], v[4 * i + 2], v[4 * i + 3]);
+                                else dst[i] = make_float4(v[4 * i], v[4 * i + 1], v[4 * i + 2], v[4 * i + 3]);
                             }
                         }
                     } else {
@@ -414,7 +446,7 @@ bool make_map(CUtensorMap *map, const void *base, uint64_t cols, uint64_t rows, 
               CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-template <int BN>
+template <int BN, int EPI>
 int launch_tc(smc_ctx *ctx, const bf16 *x, int ldx, const bf16 *w, int M, int N, int K, const smc_dense_out &o, cudaStream_t s)
 {
     using S = TcShape<BN>;
@@ -422,11 +454,11 @@ int launch_tc(smc_ctx *ctx, const bf16 *x, int ldx, const bf16 *w, int M, int N,
     if (!make_map(&mx, x, K, M, ldx, TC_M) || !make_map(&mw, w, K, N, K, BN)) return smc_fail(ctx, SMC_E_CUDA, "dense matmul: tensor map encoding failed");
     static bool attr_set = false;
     if (!attr_set) {
-        SMC_CUDA(ctx, cudaFuncSetAttribute(dense_tc_kernel<BN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)S::SMEM));
+        SMC_CUDA(ctx, cudaFuncSetAttribute(dense_tc_kernel<BN, EPI>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)S::SMEM));
         attr_set = true;
     }
     const int tiles = ((M + TC_M - 1) / TC_M) * ((N + BN - 1) / BN);
-    smc_launch_dep(ctx->use_pdl, dense_tc_kernel<BN>, dim3(tiles < ctx->sm_count ? tiles : ctx->sm_count), dim3(192), S::SMEM, s, mx, mw, M, N, K, o,
+    smc_launch_dep(ctx->use_pdl, dense_tc_kernel<BN, EPI>, dim3(tiles < ctx->sm_count ? tiles : ctx->sm_count), dim3(192), S::SMEM, s, mx, mw, M, N, K, o,
                    ctx->d_status);
     SMC_LAUNCH_CHECK(ctx);
     return SMC_OK;
@@ -471,12 +503,18 @@ int smc_launch_dense_rows(smc_ctx *ctx, const void *x, int x_bf16, int ldx, cons
     const bool vec = x_bf16 && K % 8 == 0 && ldx % 8 == 0 && aligned(x) && aligned(w);
     if (vec) {
         const bf16 *xb = static_cast<const bf16 *>(x);
-        if (M > 32 && aligned(o.y)) {
+        if (M > 32 && aligned(o.y) && aligned(o.bias)) {
             // rounds of tiles over the device: a wide tile takes less than twice as long as a narrow one
             const long long mt = (M + TC_M - 1) / TC_M, sms = ctx->sm_count;
             const long long wide = 2 * ((mt * ((N + 255) / 256) + sms - 1) / sms), narrow = (mt * ((N + 127) / 128) + sms - 1) / sms;
-            if (5 * wide <= 6 * narrow) return launch_tc<256>(ctx, xb, ldx, w, M, N, K, o, s);
-            return launch_tc<128>(ctx, xb, ldx, w, M, N, K, o, s);
+            auto tc = [&](auto epi) {
+                constexpr int E = decltype(epi)::value;
+                return 5 * wide <= 6 * narrow ? launch_tc<256, E>(ctx, xb, ldx, w, M, N, K, o, s) : launch_tc<128, E>(ctx, xb, ldx, w, M, N, K, o, s);
+            };
+            if (o.woven == 2) return tc(std::integral_constant<int, EPI_GELU_PAIRS>());
+            if (o.woven) return tc(std::integral_constant<int, EPI_SILU_PAIRS>());
+            if (o.bias || o.silu_to > o.silu_from || o.softcap > 0.f) return tc(std::integral_constant<int, EPI_FINISH>());
+            return tc(std::integral_constant<int, EPI_STORE>());
         }
         launch_skinny(ctx, xb, ldx, 0, w, 1, N, K, M, o, s);
         SMC_LAUNCH_CHECK(ctx);

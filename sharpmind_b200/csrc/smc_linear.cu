@@ -109,7 +109,8 @@ __global__ void __launch_bounds__(128) linear_step_kernel(const T *__restrict__ 
 // ------------------------------------------------------------------------------ norm in parts, then gate
 // o = y / rms(part) * w * gate(g) * out_scale; a warp (WARP) or a CTA per (row, part).  The gate's inputs were made by the
 // kernel before the predecessor and are requested before the wait.
-__device__ __forceinline__ float gate_of(int sigmoid, float g) { return sigmoid ? __fdiv_rn(1.0f, 1.0f + expf(-g)) : silu(g); }
+template <typename T> __device__ __forceinline__ float gate_of(int sigmoid, float g) { return sigmoid ? __fdiv_rn(1.0f, 1.0f + expf(-g)) : silu(g); }
+template <> __device__ __forceinline__ float gate_of<bf16>(int sigmoid, float g) { return __fdividef(sigmoid ? 1.0f : g, 1.0f + __expf(-g)); }
 
 template <typename T, int V, bool WARP>
 __global__ void __launch_bounds__(256) norm_gate_kernel(const float *__restrict__ y, const T *__restrict__ g, int ld, const float *__restrict__ w,
@@ -152,7 +153,7 @@ __global__ void __launch_bounds__(256) norm_gate_kernel(const float *__restrict_
     const float inv = __fdiv_rn(1.0f, sqrtf(__fdiv_rn(ss, (float)n) + eps));
     auto finish = [&](int i, float (&a)[V], float (&b)[V]) {
 #pragma unroll
-        for (int j = 0; j < V; ++j) a[j] = ((a[j] * inv) * (w ? w[base + i + j] : 1.0f)) * (gate_of(sigmoid, b[j]) * out_scale);
+        for (int j = 0; j < V; ++j) a[j] = ((a[j] * inv) * (w ? w[base + i + j] : 1.0f)) * (gate_of<T>(sigmoid, b[j]) * out_scale);
         store_v<T, V>(o + (size_t)r * ldo + base + i, a);
     };
 #pragma unroll
@@ -170,28 +171,35 @@ __global__ void __launch_bounds__(256) norm_gate_kernel(const float *__restrict_
 constexpr int CH = SMC_LINEAR_CHUNK, CTH = 256, PB = 64;  // tokens per chunk, threads, value columns per state CTA
 __host__ __device__ constexpr int row_ld(int n) { return (((n + 15) & ~15) + 8) * 2; }  // bytes: an odd number of 16-byte units
 
-// q and k [row, 2 heads, N] with the first rd elements rotated; a thread per pair or unrotated element
+// q and k [row, 2 heads, N] with the first rd elements rotated; a thread per V neighbouring pairs or unrotated elements
+template <int V>
 __global__ void __launch_bounds__(256) linear_rotate_kernel(const bf16 *__restrict__ in, int ld, int col, bf16 *__restrict__ qk, smc_rows rw,
                                                             const float *__restrict__ cosT, const float *__restrict__ sinT, int max_seq, int heads, int N,
                                                             int rd)
 {
     smc_grid_dep_sync();
-    const int half = rd / 2, units = N - half;
-    const long long e = (long long)blockIdx.x * 256 + threadIdx.x;
-    if (e >= (long long)rw.n * 2 * heads * units) return;
-    const int u = (int)(e % units), h = (int)(e / units % (2 * heads)), r = (int)(e / ((long long)units * 2 * heads));
+    const int half = rd / 2, units = (N - half) / V, e = blockIdx.x * 256 + threadIdx.x, r = blockIdx.y;
+    if (e >= 2 * heads * units) return;
+    const int u = e % units * V, h = e / units;
     const bf16 *src = in + (size_t)r * ld + col + (size_t)h * N;
     bf16 *dst = qk + ((size_t)r * 2 * heads + h) * N;
-    if (u >= half) {
-        dst[half + u] = src[half + u];
-        return;
+    float a[V], b[V];
+    load_v<bf16, V>(src + half + u, b);
+    if (u < half) {
+        int slot, p;
+        row_place(rw, r, slot, p);
+        const size_t ti = (size_t)min(p, max_seq - 1) * half + u;
+        float c[V], s[V];
+        load_v<bf16, V>(src + u, a);
+        load_v<float, V>(cosT + ti, c), load_v<float, V>(sinT + ti, s);
+#pragma unroll
+        for (int i = 0; i < V; ++i) {
+            const float x = __fsub_rn(__fmul_rn(a[i], c[i]), __fmul_rn(b[i], s[i]));
+            b[i] = __fadd_rn(__fmul_rn(b[i], c[i]), __fmul_rn(a[i], s[i])), a[i] = x;
+        }
+        store_v<bf16, V>(dst + u, a);
     }
-    int slot, p;
-    row_place(rw, r, slot, p);
-    const size_t ti = (size_t)min(p, max_seq - 1) * half + u;
-    const float a = to_f(src[u]), b = to_f(src[half + u]), c = cosT[ti], s = sinT[ti];
-    dst[u] = __float2bfloat16_rn(__fsub_rn(__fmul_rn(a, c), __fmul_rn(b, s)));
-    dst[half + u] = __float2bfloat16_rn(__fadd_rn(__fmul_rn(b, c), __fmul_rn(a, s)));
+    store_v<bf16, V>(dst + half + u, b);
 }
 
 // rows of a matrix -> shared memory, 16 bytes per copy, zeros from row `have` on
@@ -439,7 +447,7 @@ __global__ void __launch_bounds__(CTH, 2) linear_out_kernel(OutArgs A, smc_rows 
             if (t >= len) return;
             const __nv_bfloat162 gg = *reinterpret_cast<const __nv_bfloat162 *>(A.g + (size_t)(t0 + t) * A.ldg + h * P + c);
             *reinterpret_cast<uint32_t *>(A.o + (size_t)(t0 + t) * A.ldo + h * P + c) =
-                pack2(x * inv * w0 * gate_of(A.sigmoid, __low2float(gg)), y * inv * w1 * gate_of(A.sigmoid, __high2float(gg)));
+                pack2(x * inv * w0 * gate_of<bf16>(A.sigmoid, __low2float(gg)), y * inv * w1 * gate_of<bf16>(A.sigmoid, __high2float(gg)));
         };
         put(ta, Y[i][0], Y[i][1], ia), put(tb, Y[i][2], Y[i][3], ib);
     }
@@ -498,9 +506,12 @@ int chunks(smc_ctx *ctx, const smc_linear_dims &d, const smc_linear_bufs &b, con
     const bf16 *q = in, *k = in + H * N, *v = in + 2 * H * N;
     size_t ldq = b.ld;
     if (d.rot_dims > 0) {
-        const long long units = (long long)rw.n * 2 * H * (N - d.rot_dims / 2);
-        smc_launch_dep(ctx->use_pdl, linear_rotate_kernel, dim3((unsigned)((units + 255) / 256)), dim3(256), 0, s, static_cast<const bf16 *>(b.in), b.ld, b.col,
-                       static_cast<bf16 *>(b.qk), rw, b.cosT, b.sinT, b.max_seq, H, N, d.rot_dims);
+        const int half = d.rot_dims / 2;
+        auto rotate = [&](auto kernel, int v) {
+            smc_launch_dep(ctx->use_pdl, kernel, dim3((2 * H * ((N - half) / v) + 255) / 256, rw.n), dim3(256), 0, s, static_cast<const bf16 *>(b.in), b.ld, b.col,
+                           static_cast<bf16 *>(b.qk), rw, b.cosT, b.sinT, b.max_seq, H, N, d.rot_dims);
+        };
+        half % 4 == 0 ? rotate(linear_rotate_kernel<4>, 4) : rotate(linear_rotate_kernel<1>, 1);  // (dim and the columns are whole eights here)
         SMC_LAUNCH_CHECK(ctx);
         q = static_cast<const bf16 *>(b.qk), k = q + H * N, ldq = 2 * (size_t)H * N;
     }

@@ -19,25 +19,35 @@ namespace {
 
 constexpr float LOG2E = 1.4426950408889634f;
 
-// dst = RMSNorm(src) * w of one head by one warp (w null: a copy)
-template <typename T, typename F>
-__device__ __forceinline__ void head_norm(const T *src, const float *w, int n, float eps, F put)
+// dst = RMSNorm(src) * w of one head by one warp (w null: a copy), V elements at a time; dst2 (may be null) gets the same
+template <typename T, int V>
+__device__ __forceinline__ void head_norm(const T *src, const float *w, int n, float eps, T *dst, T *dst2 = nullptr)
 {
     const int lane = threadIdx.x & 31;
-    float inv = 1.0f;
+    float inv = 1.0f, v[V], g[V];
     if (w) {
         float ss = 0.f;
-        for (int i = lane; i < n; i += 32) {
-            const float v = to_f(src[i]);
-            ss = fmaf(v, v, ss);
+        for (int i = lane * V; i < n; i += 32 * V) {
+            load_v<T, V>(src + i, v);
+#pragma unroll
+            for (int j = 0; j < V; ++j) ss = fmaf(v[j], v[j], ss);
         }
         inv = __fdiv_rn(1.0f, sqrtf(__fdiv_rn(smc_group_sum<32>(ss), (float)n) + eps));
     }
-    for (int i = lane; i < n; i += 32) put(i, from_f<T>(w ? (to_f(src[i]) * inv) * w[i] : to_f(src[i])));
+    for (int i = lane * V; i < n; i += 32 * V) {
+        load_v<T, V>(src + i, v);
+        if (w) {
+            load_v<float, V>(w + i, g);
+#pragma unroll
+            for (int j = 0; j < V; ++j) v[j] = (v[j] * inv) * g[j];
+        }
+        store_v<T, V>(dst + i, v);
+        if (dst2) store_v<T, V>(dst2 + i, v);
+    }
 }
 
 // A warp per (row, head): queries into q, keys and values into the cache.
-template <typename T>
+template <typename T, int V>
 __global__ void __launch_bounds__(256) attn_post_kernel(const T *__restrict__ in, int ld, int col, T *__restrict__ q, T *__restrict__ cache, smc_rows rw,
                                                         const float *__restrict__ qn, const float *__restrict__ kn, int heads, int kvh, int dim,
                                                         int vdim, int ring, float eps)
@@ -48,18 +58,13 @@ __global__ void __launch_bounds__(256) attn_post_kernel(const T *__restrict__ in
     const int r = (int)(wid / units), u = (int)(wid % units);
     if (r >= rw.n) return;
     const T *src = in + (size_t)r * ld + col;
-    if (u < heads) {
-        T *dst = q + ((size_t)r * heads + u) * dim;
-        head_norm(src + u * dim, qn, dim, eps, [&](int i, T v) { dst[i] = v; });
-        return;
-    }
+    if (u < heads) return head_norm<T, V>(src + u * dim, qn, dim, eps, q + ((size_t)r * heads + u) * dim);
     int slot, p;
     row_place(rw, r, slot, p);
     const int k = (u - heads) % kvh;
     T *dst = cache + (((size_t)slot * ring + p % ring) * kvh + k) * (dim + vdim);
-    if (u < heads + kvh) head_norm(src + (size_t)(heads + k) * dim, kn, dim, eps, [&](int i, T v) { dst[i] = v; });
-    else
-        for (int i = threadIdx.x & 31; i < vdim; i += 32) dst[dim + i] = src[(size_t)(heads + kvh) * dim + k * vdim + i];
+    if (u < heads + kvh) head_norm<T, V>(src + (size_t)(heads + k) * dim, kn, dim, eps, dst);
+    else head_norm<T, V>(src + (size_t)(heads + kvh) * dim + k * vdim, nullptr, vdim, eps, dst + dim);
 }
 
 // One CTA per (head, row); the warps take every eighth key with a running maximum each and are merged at the end.
@@ -118,21 +123,21 @@ __global__ void __launch_bounds__(256) attn_rows_kernel(const T *__restrict__ q,
 // Up to 16 query heads that share a key/value head per cluster of up to eight CTAs of four warps.  A warp takes every
 // (4 * cluster)-th tile of 16 keys into a three-stage ring of its own (no CTA barrier in the loop), keeps a running
 // (maximum, sum) and its part of the weighted values; the parts meet in (distributed) shared memory.  The row's own key is
-// normed, stored and taken by the cluster's last warp.  Keys and the position are fetched BEFORE the wait for the
+// normed, stored and put into the last tile by the warp that takes it.  Keys and the position are fetched BEFORE the wait for the
 // predecessor: a kernel that is launched early is so only after every CTA of its predecessor has passed its own wait, and
 // the older keys and the positions were written before the predecessor's launch.
 constexpr int DKT = 16, DST = 3, DWP = 4, DCL = 8;
 __host__ __device__ constexpr int tile_ld(int n) { return (((n + 15) & ~15) + 8) * 2; }  // bytes: an odd number of 16-byte units
-__host__ __device__ constexpr int decode_smem(int dim, int vdim) { return 16 * tile_ld(dim) + DWP * DST * DKT * (tile_ld(dim) + tile_ld(vdim)); }
+__host__ __device__ constexpr int decode_smem(int dim, int vdim) { return 16 * tile_ld(dim) + DWP * DST * DKT * (tile_ld(dim) + tile_ld(vdim)) + 2 * (dim + vdim); }
 
-template <int VT>  // value tiles of 8 columns
+template <int VT, int V>  // value tiles of 8 columns; elements per load of the row
 __global__ void __launch_bounds__(DWP * 32)
 attn_decode_kernel(const bf16 *__restrict__ in, int ld, int col, bf16 *cache, bf16 *__restrict__ out, int ldo, smc_rows rw, const float *__restrict__ qn,
                    const float *__restrict__ kn, const float *__restrict__ bias, int bias_len, int heads, int kvh, int dim, int vdim, int ring,
                    int window, float scale, float out_scale, float eps)
 {
     extern __shared__ __align__(16) uint8_t sm_raw[];
-    __shared__ float w_m[DWP][16], w_l[DWP][16], all_m[DCL * DWP][16], all_l[DCL * DWP][16];
+    __shared__ float w_m[DWP][16], w_l[DWP][16], all_f[DCL * DWP][16];
     const int ldk = tile_ld(dim), ldv = tile_ld(vdim), d16 = (dim + 15) & ~15, row = dim + vdim;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, tg = lane & 3;
     const int G = heads / kvh, groups = (G + 15) / 16, kh = blockIdx.y / groups, grp = blockIdx.y % groups;
@@ -141,13 +146,14 @@ attn_decode_kernel(const bf16 *__restrict__ in, int ld, int col, bf16 *cache, bf
     uint8_t *mine = sm_raw + 16 * ldk + warp * DST * stage;
     const uint32_t qb = (uint32_t)__cvta_generic_to_shared(sm_raw), kb0 = (uint32_t)__cvta_generic_to_shared(mine);
     // the query rows without a head, and padding columns that no copy writes
-    const int clear = d16 != dim ? decode_smem(dim, vdim) : 16 * ldk;
+    bf16 *own = reinterpret_cast<bf16 *>(sm_raw + 16 * ldk + DWP * DST * stage);  // the row's own key and value
+    const int clear = d16 != dim ? 16 * ldk + DWP * DST * stage : 16 * ldk;
     for (int e = threadIdx.x; e < clear / 16; e += DWP * 32) reinterpret_cast<uint4 *>(sm_raw)[e] = make_uint4(0u, 0u, 0u, 0u);
     __syncthreads();
 
     int slot, p;
     row_place(rw, r, slot, p);
-    const int old = window > 0 ? min(p, window - 1) : p, lo_row = (p - old) % ring, tiles = (old + DKT - 1) / DKT;
+    const int old = window > 0 ? min(p, window - 1) : p, lo_row = (p - old) % ring, tiles = old / DKT + 1;
     bf16 *base = cache + ((size_t)slot * ring * kvh + kh) * row;
     const int cu = dim / 8, pieces = row / 8, step = cl * DWP;
     auto fetch = [&](int t, int st) {
@@ -169,9 +175,14 @@ attn_decode_kernel(const bf16 *__restrict__ in, int ld, int col, bf16 *cache, bf
     int t = warp * cl + rank;
     fetch(t, 0), fetch(t + step, 1);
     smc_grid_dep_sync();
-    for (int hh = warp; hh < nh; hh += DWP) {
-        bf16 *dst = reinterpret_cast<bf16 *>(sm_raw + hh * ldk);
-        head_norm(in + (size_t)r * ld + col + (size_t)(h0 + hh) * dim, qn, dim, eps, [&](int i, bf16 v) { dst[i] = v; });
+    const bf16 *src = in + (size_t)r * ld + col;
+    for (int hh = warp; hh < nh; hh += DWP)
+        head_norm<bf16, V>(src + (size_t)(h0 + hh) * dim, qn, dim, eps, reinterpret_cast<bf16 *>(sm_raw + hh * ldk));
+    const bool last = (tiles - 1) % step == warp * cl + rank;  // this warp takes the last tile
+    if (last) {
+        bf16 *keep = base + (size_t)(p % ring) * kvh * row;
+        head_norm<bf16, V>(src + (size_t)(heads + kh) * dim, kn, dim, eps, own, grp == 0 ? keep : nullptr);
+        head_norm<bf16, V>(src + (size_t)(heads + kvh) * dim + kh * vdim, nullptr, vdim, eps, own + dim, grp == 0 ? keep + dim : nullptr);
     }
     __syncthreads();
 
@@ -242,31 +253,18 @@ attn_decode_kernel(const bf16 *__restrict__ in, int ld, int col, bf16 *cache, bf
         fetch(t + 2 * step, st == 0 ? 2 : st - 1);
         asm volatile("cp.async.wait_group 2;" ::: "memory");
         __syncwarp();
-        take(kb0 + (uint32_t)(st * stage), min(DKT, old - t * DKT), old - t * DKT);
+        if (last && t == tiles - 1) {
+            uint8_t *kr = mine + st * stage + (old % DKT) * ldk, *vr = mine + st * stage + DKT * ldk + (old % DKT) * ldv;
+            for (int c = lane; c < pieces; c += 32)
+                *reinterpret_cast<uint4 *>(c < cu ? kr + 16 * c : vr + 16 * (c - cu)) = *reinterpret_cast<const uint4 *>(own + 8 * c);
+            __syncwarp();
+        }
+        take(kb0 + (uint32_t)(st * stage), min(DKT, old + 1 - t * DKT), old - t * DKT);
         __syncwarp();  // the stage is refilled by the next iteration's fetch
         st = st == 2 ? 0 : st + 1;
     }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncwarp();
-    if (rank == cl - 1 && warp == DWP - 1) {  // the row's own key and value
-        const bf16 *src = in + (size_t)r * ld + col + (size_t)heads * dim;
-        bf16 *keep = base + (size_t)(p % ring) * kvh * row, *ks = reinterpret_cast<bf16 *>(mine);
-        head_norm(src + kh * dim, kn, dim, eps, [&](int i, bf16 v) {
-            ks[i] = v;
-            if (grp == 0) keep[i] = v;
-        });
-        for (int e = lane; e < DKT * ldv / 16; e += 32) reinterpret_cast<uint4 *>(mine + DKT * ldk)[e] = make_uint4(0u, 0u, 0u, 0u);
-        __syncwarp();
-        bf16 *vs = reinterpret_cast<bf16 *>(mine + DKT * ldk);
-        for (int i = lane; i < vdim; i += 32) {
-            const bf16 v = src[(size_t)kvh * dim + kh * vdim + i];
-            vs[i] = v;
-            if (grp == 0) keep[dim + i] = v;
-        }
-        __syncwarp();
-        take(kb0, 1, 0);
-        __syncwarp();
-    }
     // ---- the parts: [16][vdim] fp32 over each warp's own tiles
     const int ldp = ((vdim + 15) & ~15) + 4;
     float *part = reinterpret_cast<float *>(mine);
@@ -289,21 +287,25 @@ attn_decode_kernel(const bf16 *__restrict__ in, int ld, int col, bf16 *cache, bf
         asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(f) : "r"(v) : "memory");
         return f;
     };
-    const int parts = cl * DWP;
-    for (int e = threadIdx.x; e < parts * 16; e += DWP * 32)
-        all_m[e >> 4][e & 15] = remote(&w_m[(e >> 4) % DWP][e & 15], (e >> 4) / DWP), all_l[e >> 4][e & 15] = remote(&w_l[(e >> 4) % DWP][e & 15], (e >> 4) / DWP);
-    __syncthreads();
-    if (threadIdx.x < 16) {
-        const int hh = threadIdx.x;
-        float top = -INFINITY, den = 0.f;
-        for (int k = 0; k < parts; ++k) top = fmaxf(top, all_m[k][hh]);
-        for (int k = 0; k < parts; ++k) {
-            const float f = ex2(all_m[k][hh] - top);  // a warp without a key has -inf: 0
-            den = fmaf(f, all_l[k][hh], den);
-            all_m[k][hh] = f;
+    {  // factors: eight lanes per head, each with every eighth part
+        const int hh = threadIdx.x >> 3, sub = threadIdx.x & 7, parts = cl * DWP;
+        float m[DCL * DWP / 8], l[DCL * DWP / 8], top = -INFINITY, den = 0.f;
+#pragma unroll
+        for (int i = 0; i < DCL * DWP / 8; ++i) {
+            const int k = sub + 8 * i;
+            m[i] = k < parts ? remote(&w_m[k % DWP][hh], k / DWP) : -INFINITY, l[i] = k < parts ? remote(&w_l[k % DWP][hh], k / DWP) : 0.f;
         }
+#pragma unroll
+        for (int i = 0; i < DCL * DWP / 8; ++i) top = fmaxf(top, m[i]);
+#pragma unroll
+        for (int x = 1; x < 8; x <<= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, x));
+#pragma unroll
+        for (int i = 0; i < DCL * DWP / 8; ++i) m[i] = ex2(m[i] - top), den = fmaf(m[i], l[i], den);  // a warp without a key: 0
+#pragma unroll
+        for (int x = 1; x < 8; x <<= 1) den += __shfl_xor_sync(0xffffffffu, den, x);
         const float inv = __fdiv_rn(out_scale, den);
-        for (int k = 0; k < parts; ++k) all_m[k][hh] *= inv;
+#pragma unroll
+        for (int i = 0; i < DCL * DWP / 8; ++i) all_f[sub + 8 * i][hh] = m[i] * inv;
     }
     __syncthreads();
     const int total = nh * vdim, per = (total + cl - 1) / cl, e1 = min(total, (rank + 1) * per);
@@ -311,14 +313,15 @@ attn_decode_kernel(const bf16 *__restrict__ in, int ld, int col, bf16 *cache, bf
     const float *part0 = reinterpret_cast<const float *>(sm_raw + 16 * ldk);
     for (int e = rank * per + threadIdx.x; e < e1; e += DWP * 32) {
         const int hh = e / vdim, c = e % vdim;
-        float v = 0.f;
-        for (int k = 0; k < cl; ++k) {
-            float x[DWP];
+        float v = 0.f, x[DCL][DWP];
 #pragma unroll
-            for (int w = 0; w < DWP; ++w) x[w] = remote(part0 + (size_t)w * region + hh * ldp + c, k);
+        for (int k = 0; k < DCL; ++k)
 #pragma unroll
-            for (int w = 0; w < DWP; ++w) v = fmaf(all_m[k * DWP + w][hh], x[w], v);
-        }
+            for (int w = 0; w < DWP; ++w) x[k][w] = k < cl ? remote(part0 + (size_t)w * region + hh * ldp + c, k) : 0.f;
+#pragma unroll
+        for (int k = 0; k < DCL; ++k)
+#pragma unroll
+            for (int w = 0; w < DWP; ++w) v = fmaf(all_f[k * DWP + w][hh], x[k][w], v);
         out[(size_t)r * ldo + (size_t)(h0 + hh) * vdim + c] = __float2bfloat16_rn(v);
     }
     cluster_sync();  // nobody leaves while its parts are read
@@ -486,11 +489,11 @@ __global__ void __launch_bounds__(256) expand_bias_kernel(const float *__restric
     if (e < (long long)heads * len) out[e] = table[(size_t)bucket[e % len] * heads + e / len];
 }
 
+bool whole(const void *p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
 // rows and 16-byte pieces that the tensor-core kernels can copy
 bool pieces_fit(const smc_attn_dims &d, const smc_attn_bufs &b)
 {
-    auto aligned = [](const void *p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
-    return d.dim % 8 == 0 && d.vdim % 8 == 0 && d.vdim <= 256 && b.ld % 2 == 0 && b.ldo % 2 == 0 && aligned(b.q) && aligned(b.cache) &&
+    return d.dim % 8 == 0 && d.vdim % 8 == 0 && d.vdim <= 256 && b.ld % 2 == 0 && b.ldo % 2 == 0 && whole(b.q) && whole(b.cache) &&
            (reinterpret_cast<uintptr_t>(b.o) & 3) == 0;
 }
 
@@ -507,8 +510,13 @@ template <typename T>
 int post(smc_ctx *ctx, const smc_attn_dims &d, const smc_attn_bufs &b, const smc_rows &rw, cudaStream_t s)
 {
     const long long warps = (long long)rw.n * (d.heads + 2 * d.kv_heads);
-    smc_launch_dep(ctx->use_pdl, attn_post_kernel<T>, dim3((unsigned)((warps + 7) / 8)), dim3(256), 0, s, static_cast<const T *>(b.in), b.ld, b.col,
-                   static_cast<T *>(b.q), static_cast<T *>(b.cache), rw, b.q_norm, b.k_norm, d.heads, d.kv_heads, d.dim, d.vdim, d.ring, d.eps);
+    auto go = [&](auto kernel) {
+        smc_launch_dep(ctx->use_pdl, kernel, dim3((unsigned)((warps + 7) / 8)), dim3(256), 0, s, static_cast<const T *>(b.in), b.ld, b.col,
+                       static_cast<T *>(b.q), static_cast<T *>(b.cache), rw, b.q_norm, b.k_norm, d.heads, d.kv_heads, d.dim, d.vdim, d.ring, d.eps);
+    };
+    const bool four = d.dim % 4 == 0 && d.vdim % 4 == 0 && b.ld % 4 == 0 && b.col % 4 == 0 && whole(b.in) && whole(b.q) && whole(b.cache) &&
+                      whole(b.q_norm) && whole(b.k_norm);
+    four ? go(attn_post_kernel<T, 4>) : go(attn_post_kernel<T, 1>);
     SMC_LAUNCH_CHECK(ctx);
     return SMC_OK;
 }
@@ -541,7 +549,8 @@ int decode(smc_ctx *ctx, const smc_attn_dims &d, const smc_attn_bufs &b, const s
     int cl = DCL;
     while (cl > 1 && ((long long)rw.n * groups * cl > (long long)per_sm * ctx->sm_count || cl / 2 >= most)) cl /= 2;
     return by_value_tiles(d.vdim, [&](auto vt) {
-        auto kernel = attn_decode_kernel<decltype(vt)::value>;
+        const bool four = b.ld % 4 == 0 && b.col % 4 == 0 && whole(b.in) && whole(b.q_norm) && whole(b.k_norm);
+        auto kernel = four ? attn_decode_kernel<decltype(vt)::value, 4> : attn_decode_kernel<decltype(vt)::value, 1>;
         SMC_CUDA(ctx, cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
         smc_launch_dep_cluster(ctx->use_pdl, cl, kernel, dim3(cl, groups, rw.n), dim3(DWP * 32), smem, s, static_cast<const bf16 *>(b.in), b.ld, b.col,
                                static_cast<bf16 *>(b.cache), static_cast<bf16 *>(b.o), b.ldo, rw, b.q_norm, b.k_norm, b.bias, d.bias_len, d.heads,
