@@ -232,6 +232,9 @@ int smc_launch_embed_bf16(smc_ctx *, const smc_weight *table, const int *tokens,
 // the same selection of rows through a layer norm without a bias
 int smc_launch_layernorm(smc_ctx *, const float *x, const int *rows, int first, int n_rows, const float *w, void *out, int out_bf16, int n, float eps,
                          cudaStream_t s);
+// dense matmul of the layer-normed rows x [M, K]; one row is normed inside the matmul, more go through scratch [M, K]
+int smc_launch_dense_layernorm(smc_ctx *, const float *x, const float *norm, float eps, void *scratch, int scratch_bf16, const smc_weight *, int M,
+                               const smc_dense_out &, cudaStream_t s);
 // ---- latent attention (smc_latent.cu) ----
 struct smc_latent_dims {
     int heads, dim, rot_dim, vdim, q_rank, kv_rank, window, ring;

@@ -68,10 +68,53 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1
 // wide and a row's four lanes read 64 contiguous bytes.  The first weight chunks are requested before the kernel waits
 // for its predecessor.  Grouped form (blockIdx.z = group): N rows per group, each group with its own columns of x.
 // HALF: eight weight rows per CTA (the upper half of each fragment is zero), for matrices with too few rows to fill the SMs.
-template <int NT, int U, bool HALF>
-__global__ void __launch_bounds__(256) dense_skinny_kernel(const bf16 *__restrict__ w, const bf16 *__restrict__ x, int ldx, int M, int N, int K,
-                                                           smc_dense_out o, int x_group)
+// KV > 0: one fp32 row of up to 1024 KV elements instead of x, layer-normed by every CTA while its first weights arrive.
+struct NormedRow {
+    const float *x, *w;
+    float eps;
+};
+template <int KV>
+__device__ __forceinline__ void stage_normed(const NormedRow &r, int K, bf16 *xs)
 {
+    __shared__ float red[2][8];
+    float4 v[KV], g[KV];
+    float sum = 0.f, ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < KV; ++j) {
+        const int i = threadIdx.x + 256 * j;
+        v[j] = 4 * i < K ? reinterpret_cast<const float4 *>(r.x)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+        g[j] = 4 * i < K ? __ldg(reinterpret_cast<const float4 *>(r.w) + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    auto block = [&](float t, float *s) {
+        t = smc_group_sum<32>(t);
+        if ((threadIdx.x & 31) == 0) s[threadIdx.x >> 5] = t;
+        __syncthreads();
+        return ((s[0] + s[1]) + (s[2] + s[3])) + ((s[4] + s[5]) + (s[6] + s[7]));
+    };
+#pragma unroll
+    for (int j = 0; j < KV; ++j) sum += (v[j].x + v[j].y) + (v[j].z + v[j].w);
+    const float mean = __fdiv_rn(block(sum, red[0]), (float)K);
+#pragma unroll
+    for (int j = 0; j < KV; ++j) {
+        if (4 * (threadIdx.x + 256 * j) >= K) continue;
+        v[j].x -= mean, v[j].y -= mean, v[j].z -= mean, v[j].w -= mean;
+        ss = fmaf(v[j].x, v[j].x, ss), ss = fmaf(v[j].y, v[j].y, ss), ss = fmaf(v[j].z, v[j].z, ss), ss = fmaf(v[j].w, v[j].w, ss);
+    }
+    const float inv = __fdiv_rn(1.0f, sqrtf(__fdiv_rn(block(ss, red[1]), (float)K) + r.eps));
+#pragma unroll
+    for (int j = 0; j < KV; ++j) {
+        const int i = threadIdx.x + 256 * j;
+        if (4 * i < K)
+            *reinterpret_cast<uint2 *>(xs + 4 * i) = make_uint2(pack2((v[j].x * inv) * g[j].x, (v[j].y * inv) * g[j].y),
+                                                                pack2((v[j].z * inv) * g[j].z, (v[j].w * inv) * g[j].w));
+    }
+    __syncthreads();
+}
+template <int NT, int U, bool HALF, int KV = 0>
+__global__ void __launch_bounds__(256) dense_skinny_kernel(const bf16 *__restrict__ w, const bf16 *__restrict__ x, int ldx, int M, int N, int K,
+                                                           smc_dense_out o, int x_group, NormedRow row)
+{
+    __shared__ __align__(16) bf16 xs[KV ? 1024 * KV : 8];
     constexpr int TOK = NT * 8, ROWS = HALF ? 8 : 16;
     __shared__ float red[8][ROWS][TOK + 1];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, q = lane & 3;
@@ -92,6 +135,7 @@ __global__ void __launch_bounds__(256) dense_skinny_kernel(const bf16 *__restric
     };
     fetch(warp);
     smc_grid_dep_sync();
+    if constexpr (KV > 0) stage_normed<KV>(row, K, xs);
     float acc[NT][4];
 #pragma unroll
     for (int t = 0; t < NT; ++t) acc[t][0] = acc[t][1] = acc[t][2] = acc[t][3] = 0.f;
@@ -106,7 +150,8 @@ __global__ void __launch_bounds__(256) dense_skinny_kernel(const bf16 *__restric
 #pragma unroll
             for (int t = 0; t < NT; ++t) {
                 const int m = m0 + 8 * t + g;
-                xv[u][t] = m < M && k < K ? *reinterpret_cast<const uint4 *>(x + (size_t)m * ldx + k) : zero;
+                if (KV) xv[u][t] = m == 0 && k < K ? *reinterpret_cast<const uint4 *>(xs + k) : zero;
+                else xv[u][t] = m < M && k < K ? *reinterpret_cast<const uint4 *>(x + (size_t)m * ldx + k) : zero;
             }
         }
         fetch(c0 + 8 * U);
@@ -469,12 +514,23 @@ void launch_skinny(smc_ctx *ctx, const bf16 *x, int ldx, int x_group, const bf16
     const int nt = M <= 8 ? 1 : (M <= 16 ? 2 : 4), my = (M + nt * 8 - 1) / (nt * 8);
     const bool half = (long long)((N + 15) / 16) * my * groups < 2 * ctx->sm_count;  // fewer than two CTAs per SM
     const dim3 grid(half ? (N + 7) / 8 : (N + 15) / 16, my, groups);
-    auto go = [&](auto kernel) { smc_launch_dep(ctx->use_pdl, kernel, grid, dim3(256), 0, s, w, x, ldx, M, N, K, o, x_group); };
+    auto go = [&](auto kernel) { smc_launch_dep(ctx->use_pdl, kernel, grid, dim3(256), 0, s, w, x, ldx, M, N, K, o, x_group, NormedRow{}); };
     const bool deep = K >= 2048;  // eight chunks and more per warp
     if (nt == 1 && deep) half ? go(dense_skinny_kernel<1, 8, true>) : go(dense_skinny_kernel<1, 8, false>);
     else if (nt == 1) half ? go(dense_skinny_kernel<1, 4, true>) : go(dense_skinny_kernel<1, 4, false>);
     else if (nt == 2) half ? go(dense_skinny_kernel<2, 4, true>) : go(dense_skinny_kernel<2, 4, false>);
     else half ? go(dense_skinny_kernel<4, 4, true>) : go(dense_skinny_kernel<4, 4, false>);
+}
+
+// one fp32 row, layer-normed on the way
+template <int KV, int U>
+void launch_skinny_normed(smc_ctx *ctx, const NormedRow &row, const bf16 *w, int N, int K, const smc_dense_out &o, cudaStream_t s)
+{
+    const bool half = (N + 15) / 16 < 2 * ctx->sm_count;
+    auto go = [&](auto kernel) {
+        smc_launch_dep(ctx->use_pdl, kernel, dim3(half ? (N + 7) / 8 : (N + 15) / 16), dim3(256), 0, s, w, (const bf16 *)nullptr, 0, 1, N, K, o, 0, row);
+    };
+    half ? go(dense_skinny_kernel<1, U, true, KV>) : go(dense_skinny_kernel<1, U, false, KV>);
 }
 
 __global__ void __launch_bounds__(256) round_bf16_kernel(const float *__restrict__ x, bf16 *__restrict__ y, long long n)
@@ -549,4 +605,21 @@ int smc_launch_dense_grouped(smc_ctx *ctx, const void *x, int ldx, int x_group, 
 int smc_launch_dense(smc_ctx *ctx, const void *x, int x_bf16, int ldx, const smc_weight *w, int M, const smc_dense_out &o, cudaStream_t s)
 {
     return smc_launch_dense_rows(ctx, x, x_bf16, ldx, w, 0, w->N, M, o, s);
+}
+
+int smc_launch_dense_layernorm(smc_ctx *ctx, const float *x, const float *norm, float eps, void *scratch, int scratch_bf16, const smc_weight *wt, int M,
+                               const smc_dense_out &o, cudaStream_t s)
+{
+    const int K = wt->K;
+    auto aligned = [](const void *p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+    // worth it while one wave of CTAs covers the matrix: the CTAs of a later wave would norm the row again with nothing to hide it
+    if (M == 1 && scratch_bf16 && wt->dtype == SMC_BF16 && K % 8 == 0 && K <= 1024 && (wt->N + 15) / 16 <= 3 * ctx->sm_count && aligned(x) && aligned(norm) && aligned(wt->d_raw)) {
+        const NormedRow row{x, norm, eps};
+        const bf16 *w = reinterpret_cast<const bf16 *>(wt->d_raw);
+        launch_skinny_normed<1, 4>(ctx, row, w, wt->N, K, o, s);
+        SMC_LAUNCH_CHECK(ctx);
+        return SMC_OK;
+    }
+    int rc = smc_launch_layernorm(ctx, x, nullptr, 0, M, norm, scratch, scratch_bf16, K, eps, s);
+    return rc ? rc : smc_launch_dense(ctx, scratch, scratch_bf16, K, wt, M, o, s);
 }

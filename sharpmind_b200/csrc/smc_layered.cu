@@ -314,15 +314,18 @@ int smc_layered_forward(smc_ctx *ctx, smc_layered *m, const int *d_tokens, int c
         int rc = smc_launch_dense(ctx, a, bf, k, w, n, out, s);
         return rc || before ? rc : smc_scaled_add_rmsnorm_dev(ctx, m->x, m->y, norm, m->x16, n, H, d.alpha, 1.0f, d.eps, s);
     };
-    auto prepare = [&](const float *norm) -> int { return before ? smc_launch_layernorm(ctx, m->x, nullptr, 0, n, norm, xin, bf, H, d.eps, s) : (int)SMC_OK; };
+    // a matmul over the layer's input, normed first where the norm comes before
+    auto project = [&](const float *norm, const smc_weight *w, const smc_dense_out &out) -> int {
+        if (before) return smc_launch_dense_layernorm(ctx, m->x, norm, d.eps, xin, bf, w, n, out, s);
+        return smc_launch_dense(ctx, xin, bf, H, w, n, out, s);
+    };
     for (int l = 0; l < d.n_layers; ++l) {
         const smc_layer_desc &L = m->layers[l];
         smc_layered::State &st = m->state[l];
-        SMC_TRY(prepare(L.norm1));
         if (L.mixer == SMC_MIX_LATENT) {
             const smc_latent_dims ld = latent_dims(m, l);
             const smc_latent_bufs lb{m->wide, m->cq, m->q, m->qa, m->oc, st.ukt, m->o, m->keys, m->kv, st.ring};
-            SMC_TRY(smc_launch_dense(ctx, xin, bf, H, L.w_down, n, to(m->wide, L.w_down->N, bf), s));
+            SMC_TRY(project(L.norm1, L.w_down, to(m->wide, L.w_down->N, bf)));
             SMC_TRY(smc_latent_post(ctx, ld, lb, rw, bf, L.q_norm, L.kv_norm, st.cosT, st.sinT, d.max_seq, s));
             SMC_TRY(smc_launch_dense(ctx, m->cq, bf, L.q_rank, L.w_uq, n, to(m->q, L.w_uq->N, bf), s));
             SMC_TRY(smc_latent_attend(ctx, ld, lb, rw, bf, L.w_ukv, L.sink, st.cosT, st.sinT, d.max_seq, pos, s));
@@ -331,7 +334,7 @@ int smc_layered_forward(smc_ctx *ctx, smc_layered *m, const int *d_tokens, int c
             smc_dense_out out = to(m->wide, ld, bf);
             out.bias = L.b_in;
             if (L.linear.heads && L.linear.silu) out.silu_from = lc, out.silu_to = ld - L.linear.heads * L.linear.vdim;
-            SMC_TRY(smc_launch_dense(ctx, xin, bf, H, L.w_in, n, out, s));
+            SMC_TRY(project(L.norm1, L.w_in, out));
             char *o2 = static_cast<char *>(m->o) + (size_t)L.attn.heads * L.attn.vdim * (bf ? 2 : 4);  // the linear heads' columns
             if (L.attn.heads) {
                 const smc_attn_bufs ab{m->wide, ld, 0, m->q, st.ring, m->o, ldo, L.attn.q_norm, L.attn.k_norm, st.bias};
@@ -346,7 +349,7 @@ int smc_layered_forward(smc_ctx *ctx, smc_layered *m, const int *d_tokens, int c
             const int ld = 2 * L.heads * L.vdim + 2 * L.groups * L.state;
             smc_dense_out out = to(m->wide, ld, bf);
             out.y32 = m->dt_raw, out.ld32 = L.heads, out.split = ld;  // step sizes stay fp32
-            SMC_TRY(smc_launch_dense(ctx, xin, bf, H, L.w_in, n, out, s));
+            SMC_TRY(project(L.norm1, L.w_in, out));
             const smc_ssm_bufs sb{m->wide, ld, m->dt_raw, m->xbc, m->ssm_y, m->o, st.conv, st.ssm};
             SMC_TRY(smc_ssm_mix(ctx, ssm_dims(m, L), sb, rw, bf, L.conv_w, L.conv_b, L.dt_bias, L.a_log, L.d_skip, L.mix_norm, s));
         }
@@ -354,8 +357,7 @@ int smc_layered_forward(smc_ctx *ctx, smc_layered *m, const int *d_tokens, int c
         if (L.ffn) {
             smc_dense_out out = to(m->act, L.ffn, bf);
             out.woven = d.ffn_act == SMC_FFN_GELU_TANH ? 2 : 1;
-            SMC_TRY(prepare(L.norm2));
-            SMC_TRY(smc_launch_dense(ctx, xin, bf, H, L.w_gu, n, out, s));
+            SMC_TRY(project(L.norm2, L.w_gu, out));
             SMC_TRY(join(m->act, L.ffn, L.w_ffn_down, L.norm2));
         }
         if (m->dump)
@@ -371,10 +373,14 @@ int smc_layered_forward(smc_ctx *ctx, smc_layered *m, const int *d_tokens, int c
     const int wanted = all_rows == 0 ? 1 : (all_rows == 1 ? n : n_rows);
     if (wanted == 0) return SMC_OK;
     if (wanted > m->rows) return smc_fail(ctx, SMC_E_RANGE, "layered model: %d logit rows of a pass of %d tokens", wanted, n);
-    SMC_TRY(final_norm(all_rows == 2 ? d_rows : nullptr, all_rows == 0 ? n - 1 : 0, wanted, m->head, bf));
     smc_dense_out logits = to(d_logits, d.vocab, 0);
     logits.softcap = d.softcap;
-    SMC_TRY(smc_launch_dense(ctx, m->head, bf, H, d.embedding, wanted, logits, s));
+    if (before && wanted == 1 && all_rows != 2) {
+        SMC_TRY(smc_launch_dense_layernorm(ctx, m->x + (size_t)(n - 1) * H, d.final_norm, d.eps, m->head, bf, d.embedding, 1, logits, s));
+    } else {
+        SMC_TRY(final_norm(all_rows == 2 ? d_rows : nullptr, all_rows == 0 ? n - 1 : 0, wanted, m->head, bf));
+        SMC_TRY(smc_launch_dense(ctx, m->head, bf, H, d.embedding, wanted, logits, s));
+    }
     if (d_argmax) SMC_TRY(smc_argmax_dev(ctx, d_logits, wanted, d.vocab, d_argmax, s));
 #undef SMC_TRY
     return SMC_OK;

@@ -11,6 +11,7 @@
 //   attn_rows_kernel      fp32 and odd sizes
 #include <math.h>
 
+#include <type_traits>
 #include <vector>
 
 #include "smc_mma.cuh"
@@ -65,6 +66,50 @@ __global__ void __launch_bounds__(256) attn_post_kernel(const T *__restrict__ in
     T *dst = cache + (((size_t)slot * ring + p % ring) * kvh + k) * (dim + vdim);
     if (u < heads + kvh) head_norm<T, V>(src + (size_t)(heads + k) * dim, kn, dim, eps, dst);
     else head_norm<T, V>(src + (size_t)(heads + kvh) * dim + k * vdim, nullptr, vdim, eps, dst + dim);
+}
+
+// The same for bfloat16 heads of up to 128 elements in whole eights: half a warp per head, eight heads of a row per warp.
+__global__ void __launch_bounds__(256) attn_post8_kernel(const bf16 *__restrict__ in, int ld, int col, bf16 *__restrict__ q, bf16 *__restrict__ cache,
+                                                         smc_rows rw, const float *__restrict__ qn, const float *__restrict__ kn, int heads, int kvh,
+                                                         int dim, int vdim, int ring, float eps)
+{
+    const int units = heads + 2 * kvh, per = (units + 7) / 8, sub = threadIdx.x >> 4 & 1, i = 8 * (threadIdx.x & 15);
+    float g[2][8];  // the weights of queries and keys
+#pragma unroll
+    for (int k = 0; k < 8; ++k) g[0][k] = qn && i + k < dim ? qn[i + k] : 1.f, g[1][k] = kn && i + k < dim ? kn[i + k] : 1.f;
+    smc_grid_dep_sync();
+    const int wid = blockIdx.x * 8 + (threadIdx.x >> 5), r = wid / per, u0 = wid % per * 8 + sub;
+    if (r >= rw.n) return;
+    int slot, p;
+    row_place(rw, r, slot, p);
+    const bf16 *src = in + (size_t)r * ld + col;
+    bf16 *row = cache + ((size_t)slot * ring + p % ring) * kvh * (dim + vdim);
+    uint4 raw[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+        const int u = u0 + 2 * j, v = u - heads - kvh;
+        raw[j] = make_uint4(0u, 0u, 0u, 0u);
+        if (u < units && i < (v < 0 ? dim : vdim)) raw[j] = *reinterpret_cast<const uint4 *>(v < 0 ? src + u * dim + i : src + (heads + kvh) * dim + v * vdim + i);
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+        const int u = u0 + 2 * j, v = u - heads - kvh;
+        const bool key = u >= heads;
+        const bf16 *e = reinterpret_cast<const bf16 *>(&raw[j]);
+        float x[8], ss = 0.f;
+#pragma unroll
+        for (int k = 0; k < 8; ++k) x[k] = to_f(e[k]), ss = fmaf(x[k], x[k], ss);
+#pragma unroll
+        for (int d = 1; d < 16; d <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, d);
+        if (v < 0 && (key ? kn : qn)) {
+            const float inv = rsqrtf(__fdividef(ss, (float)dim) + eps);
+#pragma unroll
+            for (int k = 0; k < 8; ++k) x[k] = (x[k] * inv) * (key ? g[1][k] : g[0][k]);
+            raw[j] = make_uint4(pack2(x[0], x[1]), pack2(x[2], x[3]), pack2(x[4], x[5]), pack2(x[6], x[7]));
+        }
+        bf16 *dst = !key ? q + ((size_t)r * heads + u) * dim : (v < 0 ? row + (u - heads) * (dim + vdim) : row + v * (dim + vdim) + dim);
+        if (u < units && i < (v < 0 ? dim : vdim)) *reinterpret_cast<uint4 *>(dst + i) = raw[j];
+    }
 }
 
 // One CTA per (head, row); the warps take every eighth key with a running maximum each and are merged at the end.
@@ -130,7 +175,9 @@ constexpr int DKT = 16, DST = 3, DWP = 4, DCL = 8;
 __host__ __device__ constexpr int tile_ld(int n) { return (((n + 15) & ~15) + 8) * 2; }  // bytes: an odd number of 16-byte units
 __host__ __device__ constexpr int decode_smem(int dim, int vdim) { return 16 * tile_ld(dim) + DWP * DST * DKT * (tile_ld(dim) + tile_ld(vdim)) + 2 * (dim + vdim); }
 
-template <int VT, int V>  // value tiles of 8 columns; elements per load of the row
+// VT: value tiles of 8 columns; HALF: up to eight heads (the other half of each fragment is not used); QS > 0: the queries'
+// fragments (16 elements each, up to QS of them) stay in registers.
+template <int VT, bool HALF, int QS>
 __global__ void __launch_bounds__(DWP * 32)
 attn_decode_kernel(const bf16 *__restrict__ in, int ld, int col, bf16 *cache, bf16 *__restrict__ out, int ldo, smc_rows rw, const float *__restrict__ qn,
                    const float *__restrict__ kn, const float *__restrict__ bias, int bias_len, int heads, int kvh, int dim, int vdim, int ring,
@@ -156,18 +203,28 @@ attn_decode_kernel(const bf16 *__restrict__ in, int ld, int col, bf16 *cache, bf
     const int old = window > 0 ? min(p, window - 1) : p, lo_row = (p - old) % ring, tiles = old / DKT + 1;
     bf16 *base = cache + ((size_t)slot * ring * kvh + kh) * row;
     const int cu = dim / 8, pieces = row / 8, step = cl * DWP;
+    const size_t pitch = (size_t)kvh * row;
     auto fetch = [&](int t, int st) {
         if (t < tiles) {
-            const uint32_t kb = kb0 + (uint32_t)(st * stage), vb = kb + (uint32_t)(DKT * ldk);
-#pragma unroll 4
-            for (int j = 0; j < DKT; ++j) {
-                const int k = t * DKT + j;
-                const bool seen = k < old;
-                int rr = lo_row + (seen ? k : 0);
-                rr -= rr >= ring ? ring : 0;  // old < ring
-                const bf16 *src = base + (size_t)rr * kvh * row;
-                for (int c = lane; c < pieces; c += 32)
-                    cp16(c < cu ? kb + (uint32_t)(j * ldk + 16 * c) : vb + (uint32_t)(j * ldv + 16 * (c - cu)), src + 8 * c, seen);
+            const uint32_t kb = kb0 + (uint32_t)(st * stage);
+            int first = lo_row + t * DKT;
+            first -= first >= ring ? ring : 0;  // old < ring
+            const bool straight = (t + 1) * DKT <= old && first + DKT <= ring;
+            for (int c = lane; c < pieces; c += 32) {
+                uint32_t dst = c < cu ? kb + (uint32_t)(16 * c) : kb + (uint32_t)(DKT * ldk + 16 * (c - cu));
+                const uint32_t ldd = c < cu ? ldk : ldv;
+                const bf16 *src = base + (size_t)first * pitch + 8 * c;
+                if (straight) {
+#pragma unroll
+                    for (int j = 0; j < DKT; ++j, dst += ldd, src += pitch) cp16(dst, src, true);
+                } else {
+#pragma unroll 1
+                    for (int j = 0; j < DKT; ++j, dst += ldd) {
+                        const bool seen = t * DKT + j < old;
+                        const int rr = first + j - (first + j >= ring ? ring : 0);
+                        cp16(dst, seen ? base + (size_t)rr * pitch + 8 * c : base, seen);
+                    }
+                }
             }
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
@@ -177,12 +234,12 @@ attn_decode_kernel(const bf16 *__restrict__ in, int ld, int col, bf16 *cache, bf
     smc_grid_dep_sync();
     const bf16 *src = in + (size_t)r * ld + col;
     for (int hh = warp; hh < nh; hh += DWP)
-        head_norm<bf16, V>(src + (size_t)(h0 + hh) * dim, qn, dim, eps, reinterpret_cast<bf16 *>(sm_raw + hh * ldk));
+        head_norm<bf16, 4>(src + (size_t)(h0 + hh) * dim, qn, dim, eps, reinterpret_cast<bf16 *>(sm_raw + hh * ldk));
     const bool last = (tiles - 1) % step == warp * cl + rank;  // this warp takes the last tile
     if (last) {
         bf16 *keep = base + (size_t)(p % ring) * kvh * row;
-        head_norm<bf16, V>(src + (size_t)(heads + kh) * dim, kn, dim, eps, own, grp == 0 ? keep : nullptr);
-        head_norm<bf16, V>(src + (size_t)(heads + kvh) * dim + kh * vdim, nullptr, vdim, eps, own + dim, grp == 0 ? keep + dim : nullptr);
+        head_norm<bf16, 4>(src + (size_t)(heads + kh) * dim, kn, dim, eps, own, grp == 0 ? keep : nullptr);
+        head_norm<bf16, 4>(src + (size_t)(heads + kvh) * dim + kh * vdim, nullptr, vdim, eps, own + dim, grp == 0 ? keep + dim : nullptr);
     }
     __syncthreads();
 
@@ -194,51 +251,70 @@ attn_decode_kernel(const bf16 *__restrict__ in, int ld, int col, bf16 *cache, bf
     const uint32_t a_off = qb + (uint32_t)(((lane & 7) + 8 * ((lane >> 3) & 1)) * ldk + 16 * (lane >> 4));
     const uint32_t k_off = (uint32_t)(((lane & 7) + 8 * (lane >> 4)) * ldk + 16 * ((lane >> 3) & 1));
     const uint32_t v_off = (uint32_t)(DKT * ldk + ((lane & 7) + 8 * ((lane >> 3) & 1)) * ldv + 16 * (lane >> 4));
+    constexpr int R = HALF ? 1 : 2;  // fragment rows in use per lane
+    uint32_t aq[QS ? QS : 1][4];
+#pragma unroll
+    for (int ks = 0; ks < QS; ++ks) {
+        aq[ks][0] = aq[ks][1] = aq[ks][2] = aq[ks][3] = 0u;
+        if (ks < d16 / 16) ldsm4(a_off + 32 * ks, aq[ks]);
+    }
     // a tile whose first n keys count, key j at distance d - j
     auto take = [&](uint32_t tile, int n, int d) {
-        float c0[2][2], c1[2][2];
+        float c[R][4];
 #pragma unroll
-        for (int i = 0; i < 2; ++i)
+        for (int h = 0; h < R; ++h)
 #pragma unroll
-            for (int j = 0; j < 2; ++j) {
-                const int dist = max(0, min(d - (8 * i + 2 * tg + j), bias_len - 1));
-                c0[i][j] = b0 ? b0[dist] * LOG2E : 0.f, c1[i][j] = b1 ? b1[dist] * LOG2E : 0.f;
+            for (int i = 0; i < 4; ++i) {
+                const float *bh = h ? b1 : b0;
+                c[h][i] = bh ? __ldg(bh + max(0, d - (8 * (i >> 1) + 2 * tg + (i & 1)))) : 0.f;  // (d < bias_len)
             }
         float s[2][4];
 #pragma unroll
         for (int i = 0; i < 2; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
-#pragma unroll 4
-        for (int ks = 0; ks < d16 / 16; ++ks) {
-            uint32_t a[4], b[4];
-            ldsm4(a_off + 32 * ks, a);
+        auto part = [&](const uint32_t (&a)[4], int ks) {
+            uint32_t b[4];
             ldsm4(tile + k_off + 32 * ks, b);
             mma_bf16(s[0], a, b[0], b[1]);
             mma_bf16(s[1], a, b[2], b[3]);
-        }
-        float t0 = -INFINITY, t1 = -INFINITY;
+        };
+        if (QS) {
 #pragma unroll
-        for (int i = 0; i < 2; ++i)
-#pragma unroll
-            for (int j = 0; j < 2; ++j) {
-                const bool in_tile = 8 * i + 2 * tg + j < n;
-                s[i][j] = in_tile ? fmaf(s[i][j], scale2, c0[i][j]) : -INFINITY;
-                s[i][2 + j] = in_tile ? fmaf(s[i][2 + j], scale2, c1[i][j]) : -INFINITY;
-                t0 = fmaxf(t0, s[i][j]), t1 = fmaxf(t1, s[i][2 + j]);
+            for (int ks = 0; ks < QS; ++ks)
+                if (ks < d16 / 16) part(aq[ks], ks);
+        } else {
+#pragma unroll 4
+            for (int ks = 0; ks < d16 / 16; ++ks) {
+                uint32_t a[4];
+                ldsm4(a_off + 32 * ks, a);
+                part(a, ks);
             }
-        t0 = fmaxf(t0, __shfl_xor_sync(0xffffffffu, t0, 1)), t0 = fmaxf(t0, __shfl_xor_sync(0xffffffffu, t0, 2));
-        t1 = fmaxf(t1, __shfl_xor_sync(0xffffffffu, t1, 1)), t1 = fmaxf(t1, __shfl_xor_sync(0xffffffffu, t1, 2));
-        const float n0 = fmaxf(m0, t0), n1 = fmaxf(m1, t1);  // finite: the first key of a tile always counts
-        const float f0 = ex2(m0 - n0), f1 = ex2(m1 - n1);
-        m0 = n0, m1 = n1;
-        uint32_t w[4];
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-            const float e0 = ex2(s[i][0] - n0), e1 = ex2(s[i][1] - n0), e2 = ex2(s[i][2] - n1), e3 = ex2(s[i][3] - n1);
-            l0 = i ? l0 + (e0 + e1) : fmaf(l0, f0, e0 + e1), l1 = i ? l1 + (e2 + e3) : fmaf(l1, f1, e2 + e3);
-            w[2 * i] = pack2(e0, e1), w[2 * i + 1] = pack2(e2, e3);
         }
+        float f[2] = {1.f, 1.f}, e[2][4] = {};
 #pragma unroll
-        for (int i = 0; i < VT; ++i) o[i][0] *= f0, o[i][1] *= f0, o[i][2] *= f1, o[i][3] *= f1;
+        for (int h = 0; h < R; ++h) {
+            float top = -INFINITY;
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                e[h][i] = fmaf(s[i >> 1][2 * h + (i & 1)], scale2, c[h][i] * LOG2E);
+                if (n < DKT) e[h][i] = 8 * (i >> 1) + 2 * tg + (i & 1) < n ? e[h][i] : -INFINITY;
+                top = fmaxf(top, e[h][i]);
+            }
+            top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 1)), top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, 2));
+            float &m = h ? m1 : m0, &l = h ? l1 : l0;
+            top = fmaxf(m, top);  // finite: the first key of a tile always counts
+            f[h] = ex2(m - top), m = top;
+#pragma unroll
+            for (int i = 0; i < 4; ++i) e[h][i] = ex2(e[h][i] - top);
+            l = fmaf(l, f[h], (e[h][0] + e[h][1]) + (e[h][2] + e[h][3]));
+        }
+        const uint32_t w[4] = {pack2(e[0][0], e[0][1]), HALF ? 0u : pack2(e[1][0], e[1][1]), pack2(e[0][2], e[0][3]), HALF ? 0u : pack2(e[1][2], e[1][3])};
+        if (__any_sync(0xffffffffu, f[0] != 1.f || f[1] != 1.f)) {
+#pragma unroll
+            for (int i = 0; i < VT; ++i) {
+                o[i][0] *= f[0], o[i][1] *= f[0];
+                if (!HALF) o[i][2] *= f[1], o[i][3] *= f[1];
+            }
+        }
 #pragma unroll
         for (int i = 0; i < VT / 2; ++i)
             if (16 * i < vdim) {
@@ -273,7 +349,7 @@ attn_decode_kernel(const bf16 *__restrict__ in, int ld, int col, bf16 *cache, bf
         const int c = 8 * n + 2 * tg;
         if (c >= vdim) continue;
         *reinterpret_cast<float2 *>(part + g * ldp + c) = make_float2(o[n][0], o[n][1]);
-        *reinterpret_cast<float2 *>(part + (g + 8) * ldp + c) = make_float2(o[n][2], o[n][3]);
+        if (!HALF) *reinterpret_cast<float2 *>(part + (g + 8) * ldp + c) = make_float2(o[n][2], o[n][3]);
     }
     l0 += __shfl_xor_sync(0xffffffffu, l0, 1), l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
     l1 += __shfl_xor_sync(0xffffffffu, l1, 1), l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
@@ -500,7 +576,6 @@ bool pieces_fit(const smc_attn_dims &d, const smc_attn_bufs &b)
 template <typename F>
 int by_value_tiles(int vdim, F go)
 {
-    if (vdim <= 32) return go(std::integral_constant<int, 4>());
     if (vdim <= 64) return go(std::integral_constant<int, 8>());
     if (vdim <= 128) return go(std::integral_constant<int, 16>());
     return go(std::integral_constant<int, 32>());
@@ -509,14 +584,21 @@ int by_value_tiles(int vdim, F go)
 template <typename T>
 int post(smc_ctx *ctx, const smc_attn_dims &d, const smc_attn_bufs &b, const smc_rows &rw, cudaStream_t s)
 {
-    const long long warps = (long long)rw.n * (d.heads + 2 * d.kv_heads);
-    auto go = [&](auto kernel) {
+    auto go = [&](auto kernel, int units) {
+        const long long warps = (long long)rw.n * units;
         smc_launch_dep(ctx->use_pdl, kernel, dim3((unsigned)((warps + 7) / 8)), dim3(256), 0, s, static_cast<const T *>(b.in), b.ld, b.col,
                        static_cast<T *>(b.q), static_cast<T *>(b.cache), rw, b.q_norm, b.k_norm, d.heads, d.kv_heads, d.dim, d.vdim, d.ring, d.eps);
     };
     const bool four = d.dim % 4 == 0 && d.vdim % 4 == 0 && b.ld % 4 == 0 && b.col % 4 == 0 && whole(b.in) && whole(b.q) && whole(b.cache) &&
                       whole(b.q_norm) && whole(b.k_norm);
-    four ? go(attn_post_kernel<T, 4>) : go(attn_post_kernel<T, 1>);
+    const int units = d.heads + 2 * d.kv_heads;
+    if constexpr (std::is_same<T, bf16>::value)
+        if (four && d.dim <= 128 && d.vdim <= 128 && d.dim % 8 == 0 && d.vdim % 8 == 0 && b.ld % 8 == 0 && b.col % 8 == 0) {
+            go(attn_post8_kernel, (units + 7) / 8);
+            SMC_LAUNCH_CHECK(ctx);
+            return SMC_OK;
+        }
+    four ? go(attn_post_kernel<T, 4>, units) : go(attn_post_kernel<T, 1>, units);
     SMC_LAUNCH_CHECK(ctx);
     return SMC_OK;
 }
@@ -548,9 +630,11 @@ int decode(smc_ctx *ctx, const smc_attn_dims &d, const smc_attn_bufs &b, const s
     const int most = ((d.window > 0 ? d.window : d.ring) + DKT * DWP - 1) / (DKT * DWP);
     int cl = DCL;
     while (cl > 1 && ((long long)rw.n * groups * cl > (long long)per_sm * ctx->sm_count || cl / 2 >= most)) cl /= 2;
+    const bool half = d.heads / d.kv_heads <= 8, reg = d.dim <= 128;
     return by_value_tiles(d.vdim, [&](auto vt) {
-        const bool four = b.ld % 4 == 0 && b.col % 4 == 0 && whole(b.in) && whole(b.q_norm) && whole(b.k_norm);
-        auto kernel = four ? attn_decode_kernel<decltype(vt)::value, 4> : attn_decode_kernel<decltype(vt)::value, 1>;
+        constexpr int VT = decltype(vt)::value;
+        auto kernel = half ? (reg ? attn_decode_kernel<VT, true, 8> : attn_decode_kernel<VT, true, 0>)
+                           : (reg ? attn_decode_kernel<VT, false, 8> : attn_decode_kernel<VT, false, 0>);
         SMC_CUDA(ctx, cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
         smc_launch_dep_cluster(ctx->use_pdl, cl, kernel, dim3(cl, groups, rw.n), dim3(DWP * 32), smem, s, static_cast<const bf16 *>(b.in), b.ld, b.col,
                                static_cast<bf16 *>(b.cache), static_cast<bf16 *>(b.o), b.ldo, rw, b.q_norm, b.k_norm, b.bias, d.bias_len, d.heads,
@@ -589,7 +673,8 @@ int smc_attn_mix(smc_ctx *ctx, const smc_attn_dims &d, const smc_attn_bufs &b, c
     if (!is_bf16) return rows<float>(ctx, d, b, rw, s);
     constexpr int MOST = 220 * 1024;
     const bool one = rw.seq0 < 0 || rw.n == 1;
-    if (pieces_fit(d, b) && one && decode_smem(d.dim, d.vdim) <= MOST) return decode(ctx, d, b, rw, s);
+    const bool fours = b.ld % 4 == 0 && b.col % 4 == 0 && whole(b.in) && whole(b.q_norm) && whole(b.k_norm);
+    if (pieces_fit(d, b) && fours && one && decode_smem(d.dim, d.vdim) <= MOST) return decode(ctx, d, b, rw, s);
     if (pieces_fit(d, b) && !one && prefill_smem(d.dim, d.vdim) <= MOST) return prefill(ctx, d, b, rw, pos0, s);
     return rows<bf16>(ctx, d, b, rw, s);
 }
