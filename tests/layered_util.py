@@ -19,6 +19,25 @@ def mamba(heads=6, vdim=8, state=24, groups=2, conv=4, norm_groups=3, ff=72):
             "mixer": {"heads": heads, "vdim": vdim, "state": state, "groups": groups, "conv": conv, "norm_groups": norm_groups}}
 
 
+def lightning(heads=3, dim=24, vdim=16, decay=None, ff=72):
+    return {"type": "lightning", "mlp": {"kind": "dense", "ff": ff} if ff else None,
+            "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "decay": decay or [1.0 - 0.6 / 4 ** i for i in range(heads)]}}
+
+
+def parallel(heads=6, kv_heads=2, dim=24, vdim=16, window=11, scale=0.3, bias_max=40, right_heads=2, right_dim=16, right_vdim=24, rot_dims=12, base=500.0,
+             decay=None, left_scale=0.8, right_scale=0.7, ff=72):
+    return {"type": "parallel", "mlp": {"kind": "dense", "ff": ff} if ff else None,
+            "mixer": {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "mask": {"size": window}, "scale": scale, "bias_max": bias_max},
+                      "right": {"heads": right_heads, "dim": right_dim, "vdim": right_vdim, "rot": {"base": base, "dims": rot_dims},
+                                "decay": decay or [1.0 - 2.0 ** (-2 - 3 * i) for i in range(right_heads)]},
+                      "left_scale": left_scale, "right_scale": right_scale}}
+
+
+def molopel(layers, width=96, vocab=160, eps=1e-5, scale=0.7, cap=12.0):
+    return {"architecture": "Molopel", "vocab": vocab, "width": width, "norm": {"eps": eps}, "embedding": {"scale": scale}, "logit_softcap": cap,
+            "layers": list(layers)}
+
+
 def share(cfg, j):
     """A copy of layer j that uses layer j's weights."""
     return dict(copy.deepcopy(cfg["layers"][j]), weights_of=j)
@@ -28,8 +47,8 @@ def config(layers, width=96, vocab=160, eps=1e-5, alpha=2.0):
     return {"architecture": "Fitodra", "vocab": vocab, "width": width, "norm": {"eps": eps}, "postln_alpha": alpha, "layers": list(layers)}
 
 
-def weights(cfg, seed=0, gain=1.0):
-    """name -> torch bfloat16 tensor, and the same numbers in float64."""
+def weights(cfg, seed=0, gain=1.0, buckets=12):
+    """name -> torch bfloat16 tensor, and the same numbers in float64.  `buckets`: rows of the distance tables."""
     import torch
 
     from sharpmind_b200 import layered
@@ -38,8 +57,13 @@ def weights(cfg, seed=0, gain=1.0):
     t16 = {}
     for name, shape in layered.tensor_shapes(layered.read_config(cfg)).items():
         last = name.split(".", 1)[-1]
+        shape = tuple(buckets if n is None else n for n in shape)
         x = rng.standard_normal(shape)
-        if len(shape) == 2 and not last.endswith("conv"):
+        if last == "mix.left.rel":
+            pass
+        elif cfg["architecture"] == "Molopel" and last.endswith(("norm", "norm1", "norm2")):
+            x = 1.0 + 0.2 * x
+        elif len(shape) == 2 and not last.endswith("conv"):
             x *= 1.0 if name == "embed" else gain / np.sqrt(shape[1])
         elif last.endswith("conv"):
             x *= 0.5
