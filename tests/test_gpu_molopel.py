@@ -31,12 +31,13 @@ def wide(t16):
 
 
 # ---------------------------------------------------------------------------------------- operations
-@pytest.mark.parametrize("n", [8, 97, 1000, 2052, 4096, 8200])
-def test_layer_norm(dev, n):
+@pytest.mark.parametrize("rows", [5, 700])
+@pytest.mark.parametrize("n", [8, 97, 1000, 2048, 2052, 4096, 6000, 8200])
+def test_layer_norm(dev, n, rows):
     import torch
 
     rng = np.random.default_rng(n)
-    x, w = rng.standard_normal((5, n)) + 3.0, 1.0 + 0.2 * rng.standard_normal(n)
+    x, w = rng.standard_normal((rows, n)) + 3.0, 1.0 + 0.2 * rng.standard_normal(n)
     xd, wd = (torch.from_numpy(a.astype(np.float32)).cuda() for a in (x, w))
     want = lo.layer_norm(x.astype(np.float32).astype(np.float64), w.astype(np.float32).astype(np.float64), 1e-3)
     got = dev.layernorm(xd, wd, 1e-3)
