@@ -104,7 +104,8 @@ def read_config(raw: dict) -> dict:
     if arch == "Fitodra":
         cfg["alpha"] = float(raw["postln_alpha"])
     else:
-        cfg.update(norm_place=NORM_BEFORE, ffn_act=FFN_GELU_TANH, embed_scale=float(raw["embedding"]["scale"]), softcap=float(raw["logit_softcap"]))
+        cfg.update(norm_place=NORM_BEFORE, ffn_act=FFN_GELU_TANH, embed_scale=float(raw["embedding"]["scale"]),
+                   softcap=float(raw["logit_softcap"] or 0.0))
     return cfg
 
 
